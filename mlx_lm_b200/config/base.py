@@ -41,6 +41,15 @@ class BaseModelArgs:
         return dataclasses.asdict(self)
 
 
+def need_keys(d, keys, what: str) -> None:
+    """One error that names every key the object ``what`` of a configuration lacks."""
+    if not isinstance(d, dict):
+        raise ConfigError(f"{what} must be an object with the keys {', '.join(keys)}")
+    missing = [k for k in keys if k not in d]
+    if missing:
+        raise ConfigError(f"{what} lacks required key(s): {', '.join(missing)}")
+
+
 def _positive_int(name: str, v) -> None:
     if isinstance(v, bool) or not isinstance(v, int) or v <= 0:
         raise ConfigError(f"config key {name!r} must be a positive integer, got {v!r}")

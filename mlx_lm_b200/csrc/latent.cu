@@ -1,7 +1,8 @@
 // Attention over a cache of latent rows (keys and values of all heads compressed into one short vector per
 // token): what stands around the attention kernel.
 //
-// latent_prepare  From a fused projection of a token, [q | down]: `down` holds R latent columns and dr columns of a
+// latent_prepare  From a token's queries and its down projection (columns of one fused projection, or rows of two
+//                 buffers where the queries come out of a product of their own): `down` holds R latent columns and dr columns of a
 //                 rotated key part that all heads share.  The latent columns are divided by their root mean square
 //                 and multiplied by a weight (c); the key part is rotated by the position; [c | rotated part | 0..]
 //                 becomes the token's row in the pages (one "head", Dh >= R + dr wide).  Of every query head
@@ -19,7 +20,7 @@
 MLXB_DEFINE_LAST_ERROR()
 
 template <typename T>
-__global__ void latent_prepare_kernel(const T* proj, int ld, int q_off, int c_off, int H, int d, int dr, int R,
+__global__ void latent_prepare_kernel(const T* queries, int ldqs, const T* proj, int ld, int q_off, int c_off, int H, int d, int dr, int R,
                                       const float* __restrict__ w, float eps, const float* __restrict__ freq,
                                       int interleaved, const int* __restrict__ positions,
                                       const int* __restrict__ token_req, const int* __restrict__ block_table,
@@ -48,14 +49,16 @@ __global__ void latent_prepare_kernel(const T* proj, int ld, int q_off, int c_of
   pdl_wait();
   pdl_trigger();
   proj = after_wait(proj);
+  queries = after_wait(queries);
   const T* row = proj + (size_t)t * ld;
+  const T* qrow = queries + (size_t)t * ldqs + q_off;
   const int half = dr / 2;
   const float fp = (float)p;
   // rotated parts: H query heads, then the shared key part
   for (int e = threadIdx.x; e < (H + 1) * half; e += blockDim.x) {
     const int hh = e / half, i = e - hh * half;
     const int lo = interleaved ? 2 * i : i, hi = interleaved ? 2 * i + 1 : i + half;
-    const T* src = hh < H ? row + q_off + (size_t)hh * (d + dr) + d : row + c_off + R;
+    const T* src = hh < H ? qrow + (size_t)hh * (d + dr) + d : row + c_off + R;
     const float u = to_f(src[lo]), v = to_f(src[hi]);
     float sn, cs;
     sincosf(fp * freq[i], &sn, &cs);
@@ -79,7 +82,8 @@ __global__ void latent_prepare_kernel(const T* proj, int ld, int q_off, int c_of
   for (int e = R + dr + threadIdx.x; e < Dh; e += blockDim.x) pool[slot + e] = from_f<T>(0.f);
 }
 
-MLXB_EXPORT int mlxb_latent_prepare(int dtype, const void* proj, int ld, int q_off, int c_off, int H, int d, int dr, int R,
+// queries: head h's columns from q_off + h * (d + dr) of rows at stride ldqs; proj: the down projection from c_off.
+MLXB_EXPORT int mlxb_latent_prepare(int dtype, const void* queries, int ldqs, const void* proj, int ld, int q_off, int c_off, int H, int d, int dr, int R,
                                     const float* w, float eps, const float* freq, int interleaved, const int* positions,
                                     const int* token_req, const int* block_table, int max_pages, int n_pages, int page,
                                     int Dh, void* pool, int write, float* q_lat, int ldq, int qhs, int n_tokens,
@@ -89,12 +93,12 @@ MLXB_EXPORT int mlxb_latent_prepare(int dtype, const void* proj, int ld, int q_o
     return mlxb_fail(MLXB_BAD_ARG, "latent_prepare: %d heads of %d + %d, %d latent columns in rows of %d", H, d, dr, R, Dh);
   const int threads = R >= 512 ? 256 : 128;
   if (dtype == MLXB_F32)
-    launch_pdl(latent_prepare_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, (const float*)proj, ld, q_off,
-               c_off, H, d, dr, R, w, eps, freq, interleaved, positions, token_req, block_table, max_pages, n_pages, page,
+    launch_pdl(latent_prepare_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, (const float*)queries, ldqs,
+               (const float*)proj, ld, q_off, c_off, H, d, dr, R, w, eps, freq, interleaved, positions, token_req, block_table, max_pages, n_pages, page,
                Dh, (float*)pool, write, q_lat, ldq, qhs, status, mscale);
   else if (dtype == MLXB_BF16)
     launch_pdl(latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream,
-               (const __nv_bfloat16*)proj, ld, q_off, c_off, H, d, dr, R, w, eps, freq, interleaved, positions, token_req,
+               (const __nv_bfloat16*)queries, ldqs, (const __nv_bfloat16*)proj, ld, q_off, c_off, H, d, dr, R, w, eps, freq, interleaved, positions, token_req,
                block_table, max_pages, n_pages, page, Dh, (__nv_bfloat16*)pool, write, q_lat, ldq, qhs, status, mscale);
   else
     return mlxb_fail(MLXB_BAD_DTYPE, "latent_prepare: dtype code %d", dtype);

@@ -6,7 +6,9 @@
 //                  of a part: the parts share one weight), is stored as it is (offset 0) or as its distance
 //                  from one (offset 1).  A gate g (activation dtype) may come in: mode 1 multiplies x by
 //                  silu(g) BEFORE the statistics, mode 2 multiplies the normed value by silu(g).
-//                  x is float32; the result has the activation dtype.  All arithmetic is float32.
+//                  x is float32 or has the activation dtype, which the result has.  No weight: the normed value as it is
+//                  (times the offset where there is one).  All arithmetic is float32.  Rows in parts of up to 512
+//                  columns (heads) take a kernel with a warp per part.
 // residual_update  x[r, :] += scale * (f1(y1[r, :]) + f2(y2[r, :])),  f_i = rmsnorm with weight w_i over the
 //                  whole row, or the identity where w_i is null; y2 may be null.  Optionally a copy of the new
 //                  row in the activation dtype is left in `cast_out` for the products that read it next.
@@ -16,8 +18,8 @@ MLXB_DEFINE_LAST_ERROR()
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
 
-template <typename TO>
-__global__ void rmsnorm_kernel(const float* x, int ldx, const int* __restrict__ rows, int n_src_rows,
+template <typename TI, typename TO>
+__global__ void rmsnorm_kernel(const TI* x, int ldx, const int* __restrict__ rows, int n_src_rows,
                                const float* __restrict__ w, float offset, int period, const TO* gate, int ldg,
                                int gate_mode, TO* __restrict__ out, int ldo, int D, int groups, float eps) {
   __shared__ float red[33];
@@ -33,25 +35,96 @@ __global__ void rmsnorm_kernel(const float* x, int ldx, const int* __restrict__ 
     for (int c = threadIdx.x; c < Dg; c += blockDim.x) o[c] = from_f<TO>(0.f);
     return;
   }
-  const float* xr = x + (size_t)src * ldx + (size_t)g * Dg;
+  const TI* xr = x + (size_t)src * ldx + (size_t)g * Dg;
   const TO* gr = gate ? gate + (size_t)src * ldg + (size_t)g * Dg : nullptr;
   float s = 0.f;
   for (int c = threadIdx.x; c < Dg; c += blockDim.x) {
-    float v = xr[c];
+    float v = to_f(xr[c]);
     if (gate_mode == 1) v *= silu_f(to_f(gr[c]));
     s = fmaf(v, v, s);
   }
   const float rinv = 1.f / sqrtf(block_sum(s, red) / (float)Dg + eps);
   for (int c = threadIdx.x; c < Dg; c += blockDim.x) {
-    float v = xr[c];
+    float v = to_f(xr[c]);
     if (gate_mode == 1) v *= silu_f(to_f(gr[c]));
-    v = v * rinv * (offset + w[(g * Dg + c) % period]);
+    v = v * rinv * (w ? offset + w[(g * Dg + c) % period] : offset);
     if (gate_mode == 2) v *= silu_f(to_f(gr[c]));
     o[c] = from_f<TO>(v);
   }
 }
 
-MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, const float* x, int ldx, const int* rows, int n_src_rows, const float* w,
+// Four neighbouring columns: 16 bytes of float32, 8 of bfloat16.
+__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
+  const float4 q = *reinterpret_cast<const float4*>(p);
+  v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  v[0] = __uint_as_float(q.x << 16);
+  v[1] = __uint_as_float(q.x & 0xffff0000u);
+  v[2] = __uint_as_float(q.y << 16);
+  v[3] = __uint_as_float(q.y & 0xffff0000u);
+}
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&a), *reinterpret_cast<const unsigned*>(&b));
+}
+
+// Rows in several parts of at most 128 * RP_STEPS columns (a multiple of 4, accesses of four columns): a warp per part,
+// the part in registers between the sum and the result.
+constexpr int RP_STEPS = 4;
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256)
+rmsnorm_parts_kernel(const TI* x, int ldx, const float* __restrict__ w, float offset, int period, const TO* gate, int ldg,
+                     int gate_mode, TO* __restrict__ out, int ldo, int R, int Dg, int groups, float eps) {
+  pdl_wait();
+  pdl_trigger();
+  x = after_wait(x);
+  gate = after_wait(gate);
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (item >= (long long)R * groups) return;
+  const int r = (int)(item / groups), g = (int)(item - (long long)r * groups);
+  const TI* xr = x + (size_t)r * ldx + (size_t)g * Dg;
+  const TO* gr = gate_mode ? gate + (size_t)r * ldg + (size_t)g * Dg : nullptr;
+  float v[RP_STEPS][4], gv[RP_STEPS][4];
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < RP_STEPS; ++i) {
+    const int c = (i * 32 + lane) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[i][e] = gv[i][e] = 0.f;
+    if (c < Dg) {
+      load4(xr + c, v[i]);
+      if (gate_mode) load4(gr + c, gv[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < RP_STEPS; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (gate_mode == 1) v[i][e] *= silu_f(gv[i][e]);
+      s = fmaf(v[i][e], v[i][e], s);
+    }
+  const float rinv = 1.f / sqrtf(warp_sum(s) / (float)Dg + eps);
+  TO* o = out + (size_t)r * ldo + (size_t)g * Dg;
+#pragma unroll
+  for (int i = 0; i < RP_STEPS; ++i) {
+    const int c = (i * 32 + lane) * 4;
+    if (c >= Dg) continue;
+    float res[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      res[e] = v[i][e] * rinv * (w ? offset + w[(g * Dg + c + e) % period] : offset);
+      if (gate_mode == 2) res[e] *= silu_f(gv[i][e]);
+    }
+    store4(o + c, res);
+  }
+}
+
+// x_f32: x is float32 (else it has out_dtype); w may be null (the offset is then the factor).
+MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, int x_f32, const void* x, int ldx, const int* rows, int n_src_rows, const float* w,
                              float offset, int period, const void* gate, int ldg, int gate_mode, void* out, int ldo,
                              int R, int D, int groups, float eps, cudaStream_t stream) {
   if (R <= 0) return 0;
@@ -61,17 +134,18 @@ MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, const float* x, int ldx, const int* 
   if (gate_mode < 0 || gate_mode > 2 || ((gate_mode != 0) != (gate != nullptr)))
     return mlxb_fail(MLXB_BAD_ARG, "rmsnorm: gate mode %d %s a gate", gate_mode, gate ? "with" : "without");
   if (groups > 65535) return mlxb_fail(MLXB_BAD_ARG, "rmsnorm: %d parts", groups);
+  if (out_dtype != MLXB_F32 && out_dtype != MLXB_BF16) return mlxb_fail(MLXB_BAD_DTYPE, "rmsnorm: dtype code %d", out_dtype);
   const int Dg = D / groups;
-  const int threads = Dg >= 2048 ? 256 : (Dg >= 512 ? 128 : (Dg >= 128 ? 64 : 32));
-  const dim3 grid(R, groups);
-  if (out_dtype == MLXB_F32)
-    launch_pdl(rmsnorm_kernel<float>, grid, dim3(threads), 0, stream, x, ldx, rows, n_src_rows, w, offset, period,
-               (const float*)gate, ldg, gate_mode, (float*)out, ldo, D, groups, eps);
-  else if (out_dtype == MLXB_BF16)
-    launch_pdl(rmsnorm_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, x, ldx, rows, n_src_rows, w, offset,
-               period, (const __nv_bfloat16*)gate, ldg, gate_mode, (__nv_bfloat16*)out, ldo, D, groups, eps);
-  else
-    return mlxb_fail(MLXB_BAD_DTYPE, "rmsnorm: dtype code %d", out_dtype);
+  const int xb = (x_f32 || out_dtype == MLXB_F32) ? 16 : 8, ob = out_dtype == MLXB_F32 ? 16 : 8;   // bytes of four columns
+  const bool parts = groups > 1 && rows == nullptr && Dg % 4 == 0 && Dg <= 128 * RP_STEPS && ldx % 4 == 0 && ldo % 4 == 0 &&
+                     (!gate || ldg % 4 == 0) && (uintptr_t)x % xb == 0 && ((uintptr_t)out | (uintptr_t)gate) % ob == 0;
+  const int threads = parts ? 256 : (Dg >= 2048 ? 256 : (Dg >= 512 ? 128 : (Dg >= 128 ? 64 : 32)));
+  const dim3 grid = parts ? dim3((unsigned)(((long long)R * groups + 7) / 8)) : dim3(R, groups);
+#define RMS_GO(TI, TO)                                                                                                  if (parts)                                                                                                              launch_pdl(rmsnorm_parts_kernel<TI, TO>, grid, dim3(threads), 0, stream, (const TI*)x, ldx, w, offset, period,                   (const TO*)gate, ldg, gate_mode, (TO*)out, ldo, R, Dg, groups, eps);                                     else                                                                                                                    launch_pdl(rmsnorm_kernel<TI, TO>, grid, dim3(threads), 0, stream, (const TI*)x, ldx, rows, n_src_rows, w, offset,                period, (const TO*)gate, ldg, gate_mode, (TO*)out, ldo, D, groups, eps)
+  if (out_dtype == MLXB_F32) { RMS_GO(float, float); }
+  else if (x_f32) { RMS_GO(float, __nv_bfloat16); }
+  else { RMS_GO(__nv_bfloat16, __nv_bfloat16); }
+#undef RMS_GO
   return mlxb_check_launch("rmsnorm");
 }
 

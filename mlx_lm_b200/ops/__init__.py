@@ -210,6 +210,36 @@ def embed_pos(tokens, positions, wte, wpe, out, status, stream, scale: float = 1
           _p(freq), stream)
 
 
+def embed_pairs(tokens, positions, token_req, req_first_token, slots, table, pairs, last, weight, out, n_streams: int,
+                status, stream, scale: float = 1.0, buckets: int = 0, mul_prev: int = 0, mul_cur: int = 0,
+                eps: float = 0.0) -> None:
+    """``out[t, s] = rmsnorm(table[tok] * scale + pairs[row]) * weight`` for each of ``n_streams`` streams ``s`` (``out``
+    float32 ``[T, n_streams * width]``), ``row = (prev * mul_prev + tok * mul_cur) % buckets``, or the last row of ``pairs``
+    (``[buckets + 1, width]``; None: no such table) at position 0.  ``last``: float32 ``[slots, 1]``, every request's last token,
+    read for the first row a request brings and brought up to date.  ``weight`` None: no norm."""
+    for t, what in ((tokens, "tokens"), (positions, "positions"), (token_req, "token_req"), (slots, "slots"),
+                    (req_first_token, "req_first_token")):
+        _need(t, torch.int32, "embed_pairs " + what)
+    _need(out, torch.float32, "embed_pairs out")
+    T, D = out.shape[0], table.shape[1]
+    if out.shape[1] != n_streams * D or not out.is_contiguous() or not table.is_contiguous():
+        raise KernelError(f"embed_pairs: out {tuple(out.shape)} for {n_streams} streams of {D}")
+    if pairs is not None:
+        _need(pairs, table.dtype, "embed_pairs pairs")
+        _need(last, torch.float32, "embed_pairs last")
+        if pairs.shape != (buckets + 1, D) or not pairs.is_contiguous() or last.numel() != last.shape[0]:
+            raise KernelError(f"embed_pairs: pairs {tuple(pairs.shape)} for {buckets} buckets of width {D}")
+    if weight is not None:
+        _need(weight, torch.float32, "embed_pairs weight")
+        if weight.numel() != D:
+            raise KernelError(f"embed_pairs: weight of {weight.numel()} for width {D}")
+    _call("embed", "mlxb_embed_pairs", [c_int] + [c_void_p] * 10 + [c_int] * 4 + [c_float] + [ctypes.c_longlong] * 3
+          + [c_float, c_void_p, c_void_p],
+          dtype_code(table.dtype), _p(tokens), _p(positions), _p(token_req), _p(req_first_token), _p(slots), _p(table),
+          _p(pairs), _p(last), _p(weight), _p(out), T, D, table.shape[0], int(n_streams), float(scale), int(buckets),
+          int(mul_prev), int(mul_cur), float(eps), _p(status), stream)
+
+
 def gather_tokens(src, index, dst, status, stream) -> None:
     """``dst[i] = src[index[i]]`` where ``index[i] >= 0`` (int32 all): tokens a step has just sampled, handed
     to the next step on the device."""
@@ -752,7 +782,7 @@ def process_logits(logits, params, context, bias_index, bias_value, stream) -> N
 # --------------------------------------------------------------------------
 # root-mean-square norms and a float32 residual stream (csrc/rms.cu)
 
-_RMS_ARGS = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_int,
+_RMS_ARGS = [c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_int,
              c_int, c_int, c_int, c_float, c_void_p]
 
 GATE_NONE, GATE_BEFORE, GATE_AFTER = 0, 1, 2
@@ -760,18 +790,22 @@ GATE_NONE, GATE_BEFORE, GATE_AFTER = 0, 1, 2
 
 def rmsnorm(x, weight, out, eps: float, stream, offset: float = 0.0, groups: int = 1, period: Optional[int] = None,
             gate=None, gate_mode: int = GATE_NONE, rows=None) -> None:
-    """``out[r] = x[r] / sqrt(mean(x[r]^2) + eps) * (offset + weight)`` over float32 rows, the row cut into
-    ``groups`` equal parts that are normed each by itself; ``weight`` (float32) repeats every ``period`` columns
-    (default: the width).  ``gate`` (``out``'s dtype, the shape of ``x``): ``GATE_BEFORE`` multiplies ``x`` by
+    """``out[r] = x[r] / sqrt(mean(x[r]^2) + eps) * (offset + weight)`` over rows in float32 or ``out``'s dtype, the row
+    cut into ``groups`` equal parts that are normed each by itself; ``weight`` (float32) repeats every ``period`` columns
+    (default: the width); None: no weight.  ``gate`` (``out``'s dtype, the shape of ``x``): ``GATE_BEFORE`` multiplies ``x`` by
     ``silu(gate)`` before the statistics, ``GATE_AFTER`` multiplies the normed value.  ``rows``: int32 indices of
     the input rows to take."""
-    _need(x, torch.float32, "rmsnorm x")
-    _need(weight, torch.float32, "rmsnorm weight")
+    if x.dtype != out.dtype:
+        _need(x, torch.float32, "rmsnorm x")
     R, D = out.shape
     period = D if period is None else int(period)
-    if x.shape[1] != D or weight.numel() != period or D % groups:
-        raise KernelError(f"rmsnorm: x {tuple(x.shape)}, weight of {weight.numel()} every {period}, {groups} parts, "
-                          f"out {tuple(out.shape)}")
+    if weight is None:
+        offset = offset or 1.0
+    else:
+        _need(weight, torch.float32, "rmsnorm weight")
+    if x.shape[1] != D or (weight is not None and weight.numel() != period) or D % groups:
+        raise KernelError(f"rmsnorm: x {tuple(x.shape)}, weight of {weight.numel() if weight is not None else 0} every "
+                          f"{period}, {groups} parts, out {tuple(out.shape)}")
     if rows is not None:
         _need(rows, torch.int32, "rmsnorm rows")
         if rows.numel() != R:
@@ -786,7 +820,7 @@ def rmsnorm(x, weight, out, eps: float, stream, offset: float = 0.0, groups: int
         ldg = _rows(gate, "rmsnorm gate")
     elif gate_mode != GATE_NONE:
         raise KernelError("rmsnorm: a gate mode without a gate")
-    _call("rms", "mlxb_rmsnorm", _RMS_ARGS, dtype_code(out.dtype), _p(x), _rows(x, "rmsnorm x"), _p(rows), x.shape[0],
+    _call("rms", "mlxb_rmsnorm", _RMS_ARGS, dtype_code(out.dtype), int(x.dtype == torch.float32), _p(x), _rows(x, "rmsnorm x"), _p(rows), x.shape[0],
           _p(weight), float(offset), period, _p(gate), ldg, gate_mode, _p(out), _rows(out, "rmsnorm out"), R, D,
           groups, float(eps), stream)
 
@@ -834,6 +868,55 @@ def head_difference(a, rep: int, value_dim: int, lam: float, eps: float, post: f
                                           c_void_p, c_int, c_int, c_void_p],
           dtype_code(out.dtype), _p(a), _rows(a, "head_difference a"), _p(token_req), n // value_dim, int(rep),
           int(value_dim), float(lam), float(eps), float(post), _p(out), _rows(out, "head_difference out"), T, stream)
+
+
+# --------------------------------------------------------------------------
+# a residual of several streams (csrc/streams.cu)
+
+def streams_read(x, n_streams: int, w_in, weight, out, eps: float, stream, rows=None) -> None:
+    """``out[r] = rmsnorm(sum_s w_in[s] x[r, s]) * weight``: what a sublayer reads of a residual of ``n_streams`` streams
+    (``x`` float32 ``[T, n_streams * width]``).  ``rows``: int32 indices of the input rows to take."""
+    _need(x, torch.float32, "streams_read x")
+    _need(w_in, torch.float32, "streams_read in")
+    _need(weight, torch.float32, "streams_read weight")
+    R, D = out.shape
+    if x.shape[1] != n_streams * D or w_in.numel() != n_streams or weight.numel() != D:
+        raise KernelError(f"streams_read: x {tuple(x.shape)}, out {tuple(out.shape)}, {n_streams} streams")
+    if rows is not None:
+        _need(rows, torch.int32, "streams_read rows")
+    if (rows.numel() if rows is not None else x.shape[0]) != R:
+        raise KernelError(f"streams_read: {R} output rows")
+    _call("streams", "mlxb_streams_read", [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float,
+                                           c_void_p, c_int, c_int, c_int, c_void_p],
+          dtype_code(out.dtype), _p(x), _rows(x, "streams_read x"), _p(rows), x.shape[0], int(n_streams), _p(w_in), _p(weight),
+          float(eps), _p(out), _rows(out, "streams_read out"), R, D, stream)
+
+
+def streams_update(x, y, n_streams: int, mix, w_out, stream, token_req=None, nxt=None, next_out=None, eps: float = 0.0) -> None:
+    """In place on a residual of several streams: ``x_t <- sum_s mix[s, t] x_s + w_out[t] y`` (all from the old streams).
+    With ``nxt = (w_in, weight)`` and ``next_out`` (the run's dtype, ``[T, width]``), ``streams_read`` of the new rows in
+    the same pass.  Rows whose ``token_req`` is negative are left alone."""
+    _need(x, torch.float32, "streams_update x")
+    _need(y, torch.float32, "streams_update y")
+    _need(mix, torch.float32, "streams_update mix")
+    _need(w_out, torch.float32, "streams_update out")
+    T, D = y.shape
+    S = int(n_streams)
+    if x.shape != (T, S * D) or mix.shape != (S, S) or not mix.is_contiguous() or w_out.numel() != S:
+        raise KernelError(f"streams_update: x {tuple(x.shape)}, y {tuple(y.shape)}, mix {tuple(mix.shape)}, {S} streams")
+    w_in = weight = None
+    if nxt is not None:
+        w_in, weight = nxt
+        _need(w_in, torch.float32, "streams_update in")
+        _need(weight, torch.float32, "streams_update weight")
+        if next_out is None or next_out.shape != (T, D) or w_in.numel() != S or weight.numel() != D:
+            raise KernelError(f"streams_update: what reads the streams next does not fit {S} streams of {D}")
+    _call("streams", "mlxb_streams_update", [c_int, c_void_p, c_int, c_void_p, c_int, c_int] + [c_void_p] * 5
+          + [c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+          dtype_code(next_out.dtype) if nxt is not None else F32, _p(x), _rows(x, "streams_update x"), _p(y),
+          _rows(y, "streams_update y"), S, _p(mix), _p(w_out), _p(token_req), _p(w_in), _p(weight), float(eps),
+          _p(next_out) if nxt is not None else None, _rows(next_out, "streams_update next") if nxt is not None else 0, T, D,
+          stream)
 
 
 # --------------------------------------------------------------------------
@@ -917,6 +1000,61 @@ def gated_delta_scan(qkv, q_off: int, k_off: int, v_off: int, b_raw, a_raw, dt_b
           q_off, k_off, v_off, _p(b_raw), _rows(b_raw, "gated_delta b"), _p(a_raw), _rows(a_raw, "gated_delta a"),
           _p(dt_bias), _p(a_log), _p(state), _p(slots), _p(token_req), _p(req_first_token), _p(o),
           _rows(o, "gated_delta o"), H, n_key_heads, K, V, slots.numel(), stream)
+
+
+# --------------------------------------------------------------------------
+# linear attention with a fixed decay (csrc/retention.cu) and the real-gated linear recurrent unit (csrc/rglru.cu)
+
+def retention_scan(qkv, q_off: int, k_off: int, v_off: int, freq, kscale: float, decay, state, slots, positions, token_req,
+                   req_first_token, o, n_heads: int, stream, max_run: int = 0) -> None:
+    """Per (request, head): ``S <- decay S + k_t v_t^T; o_t = S^T q_t``, q and k turned by the position first (pairs
+    ``(i, i + len(freq))``; ``freq`` float32 or None), k then times ``kscale``.  ``qkv [T, .]`` holds q, k, v from the given
+    column offsets; ``decay`` float32 ``[heads]``; ``state`` float32 ``[slots, heads, V, K]`` (a head's ``K x V`` state column
+    by column); ``o`` float32 ``[T, heads*V]``.  ``max_run`` > 0: requests that bring more rows are passed over."""
+    _need(state, torch.float32, "retention_scan state")
+    _need(o, torch.float32, "retention_scan o")
+    _need(decay, torch.float32, "retention_scan decay")
+    _, H, V, K = state.shape
+    if H != n_heads or o.shape[1] != H * V or not state.is_contiguous() or decay.numel() != H:
+        raise KernelError(f"retention_scan: state {tuple(state.shape)} for {n_heads} heads, o {tuple(o.shape)}, "
+                          f"{decay.numel()} decays")
+    half = 0
+    if freq is not None:
+        _need(freq, torch.float32, "retention_scan freq")
+        half = freq.numel()
+    _call("retention", "mlxb_retention_scan", [c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float]
+          + [c_void_p] * 7 + [c_int] * 6 + [c_void_p],
+          dtype_code(qkv.dtype), _p(qkv), _rows(qkv, "retention_scan qkv"), q_off, k_off, v_off, _p(freq), half, float(kscale),
+          _p(decay), _p(state), _p(slots), _p(positions), _p(token_req), _p(req_first_token), _p(o),
+          _rows(o, "retention_scan o"), H, K, V, slots.numel(), int(max_run), stream)
+
+
+def rglru_scan(gates, r_bias, i_bias, decay, u, y, state, slots, token_req, req_first_token, out, block: int, stream,
+               singles: bool = True, portions: bool = True) -> None:
+    """Per channel: ``S <- a S + sqrt(1 - a^2) i u`` and ``out = S * gelu_tanh(y)`` with ``r``, ``i`` the sigmoids of the
+    products in ``gates`` (float32 ``[T, 2 W]``: per block of ``block`` channels the recurrence gate's, then the input
+    gate's) plus their biases, ``log a = r * decay`` (``decay`` float32 ``[W]``: ``-8 softplus(lam)``).  ``u``, ``y``,
+    ``out``: ``[T, W]`` in the run's dtype; ``state`` float32 ``[slots, W]``.  ``singles`` / ``portions``: whether requests
+    with one row / several rows are among the step's (a launch each)."""
+    _need(gates, torch.float32, "rglru_scan gates")
+    _need(state, torch.float32, "rglru_scan state")
+    T, W = out.shape
+    for t, what in ((u, "u"), (y, "y")):
+        _need(t, out.dtype, "rglru_scan " + what)
+        if t.shape != (T, W):
+            raise KernelError(f"rglru_scan: {what} {tuple(t.shape)} for out {tuple(out.shape)}")
+    for t, what in ((r_bias, "bias"), (i_bias, "bias"), (decay, "decay")):
+        _need(t, torch.float32, "rglru_scan " + what)
+        if t.numel() != W or not t.is_contiguous():
+            raise KernelError(f"rglru_scan: {what} of {t.numel()} for {W} channels")
+    if gates.shape != (T, 2 * W) or state.shape[1:] != (W,) or not state.is_contiguous():
+        raise KernelError(f"rglru_scan: gates {tuple(gates.shape)}, state {tuple(state.shape)} for {W} channels")
+    _call("rglru", "mlxb_rglru_scan", [c_int, c_void_p, c_int] + [c_void_p] * 4 + [c_int, c_void_p, c_int] + [c_void_p] * 5
+          + [c_int] * 6 + [c_void_p],
+          dtype_code(out.dtype), _p(gates), _rows(gates, "rglru_scan gates"), _p(r_bias), _p(i_bias), _p(decay), _p(u),
+          _rows(u, "rglru_scan u"), _p(y), _rows(y, "rglru_scan y"), _p(state), _p(slots), _p(token_req),
+          _p(req_first_token), _p(out), _rows(out, "rglru_scan out"), W, int(block), slots.numel(), int(bool(singles)),
+          int(bool(portions)), stream)
 
 
 # --------------------------------------------------------------------------
@@ -1125,18 +1263,21 @@ def attention_wide_step(ctx, q, q_head_stride: int, cache_k, cache_v, block_tabl
 # --------------------------------------------------------------------------
 # attention over latent rows: what stands around it (csrc/latent.cu)
 
-_LATP_ARGS = [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p,
+_LATP_ARGS = [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p,
               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
               c_float, c_void_p]
 
 
 def latent_prepare(proj, q_off: int, c_off: int, n_heads: int, dim: int, rot_dim: int, rank: int, norm_weight, eps: float,
                    freq, interleaved: bool, positions, token_req, block_table, pool, write: bool, q_lat,
-                   q_head_stride: int, status, stream, mscale: float = 1.0) -> None:
+                   q_head_stride: int, status, stream, mscale: float = 1.0, queries=None) -> None:
     """From ``proj [T, .]`` holding ``q`` (``n_heads`` heads of ``[dim | rot_dim]`` from ``q_off``) and the down
     projection (``rank + rot_dim`` columns from ``c_off``): the token's latent row ``[rmsnorm(c) * weight | rotated
     key part | 0..]`` into ``pool [n_pages, 1, page, row]``, and every head's rotated query part, float32, into
-    columns ``rank ..`` of its ``q_head_stride`` columns of ``q_lat``.  ``mscale``: a factor on every cosine and sine."""
+    columns ``rank ..`` of its ``q_head_stride`` columns of ``q_lat``.  ``mscale``: a factor on every cosine and sine.  ``queries``: the
+    tensor the query heads lie in (from ``q_off``), where they are not columns of ``proj``."""
+    if queries is None:
+        queries = proj
     n_pages, one, page, Dh = pool.shape
     _need(proj, pool.dtype, "latent_prepare proj")
     _need(q_lat, torch.float32, "latent_prepare q_lat")
@@ -1147,7 +1288,11 @@ def latent_prepare(proj, q_off: int, c_off: int, n_heads: int, dim: int, rot_dim
         _need(freq, torch.float32, "latent_prepare freq")
         if freq.numel() != rot_dim // 2:
             raise KernelError(f"latent_prepare: {freq.numel()} frequencies for {rot_dim} rotated dimensions")
-    _call("latent", "mlxb_latent_prepare", _LATP_ARGS, dtype_code(pool.dtype), _p(proj), _rows(proj, "latent_prepare proj"),
+    _need(queries, pool.dtype, "latent_prepare queries")
+    if queries.shape[0] != proj.shape[0] or q_off + n_heads * (dim + rot_dim) > queries.shape[1]:
+        raise KernelError(f"latent_prepare: queries {tuple(queries.shape)} for {n_heads} heads of {dim} + {rot_dim}")
+    _call("latent", "mlxb_latent_prepare", _LATP_ARGS, dtype_code(pool.dtype), _p(queries),
+          _rows(queries, "latent_prepare queries"), _p(proj), _rows(proj, "latent_prepare proj"),
           q_off, c_off, n_heads, dim, rot_dim, rank, _p(norm_weight), float(eps), _p(freq), int(bool(interleaved)),
           _p(positions), _p(token_req), _p(block_table), block_table.shape[1], n_pages, page, Dh, _p(pool),
           int(bool(write)), _p(q_lat), _rows(q_lat, "latent_prepare q_lat"), q_head_stride, proj.shape[0], _p(status),

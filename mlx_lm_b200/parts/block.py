@@ -11,7 +11,7 @@ from typing import Optional
 import torch
 
 from .. import ops
-from .base import Block, FeedForward, Mixer, Norm, register_part
+from .base import VECTOR, Block, FeedForward, Init, Mixer, Norm, ParamSpec, register_part
 
 # In bfloat16 a block lets its mixer and its feed-forward fold the norm before them into their first linear
 # layer (parts/linear.py, ``Linear.fold_norm``): steps of few rows then run no norm kernels inside the blocks.
@@ -165,6 +165,105 @@ class SandwichBlock(Block):
         return x
 
 
+class HyperBlock(Block):
+    """A pre-norm block over several float32 residual streams (hyper-connections), ``x`` being ``[x_1 | .. | x_S]``.  Around
+    each sublayer ``q`` (1: the mixer, 2: the feed-forward, if the layer has one):
+    ``y = sublayer(norm_q(sum_s in_q[s] x_s))``, then, all streams from the old ones,
+    ``x_t <- sum_s mix_q[s, t] x_s + residual_scale * out_q[t] y`` (``<name>.hc<q>.in``, ``.out``, ``.mix``, float32).
+    ``learned=False``: no such tensors; ``in``, ``out`` and ``mix`` are 1 (one stream: an ordinary residual sum with a factor).
+
+    The sublayers leave their results in float32 (``mixer.mix``, ``feed_forward.branch`` with one row a token), and one
+    kernel does the streams' update together with what reads them next: the weighted sum and the norm of this block's
+    second sublayer, or of the block that runs next (``ctx.next_block``), whose input then waits in ``ctx.carried``.  The
+    norms are RMS norms (``Norm.rms_args()``)."""
+    replayable = True
+    kernel_libs = ("streams",)
+
+    def __init__(self, name: str, n_streams: int, norm_1: Norm, mixer: Mixer, norm_2: Optional[Norm] = None,
+                 feed_forward: Optional[FeedForward] = None, residual_scale: float = 1.0, learned: bool = True):
+        if (norm_2 is None) != (feed_forward is None):
+            raise ValueError("a feed-forward and the norm before it come together")
+        if not learned and n_streams != 1:
+            raise ValueError(f"{name}: {n_streams} streams need tensors that say how they are read and mixed")
+        if not 1 <= n_streams <= 16:
+            raise ValueError(f"{name}: {n_streams} residual streams (1 to 16)")
+        self.name, self.n_streams, self.residual_scale, self.learned = name, int(n_streams), float(residual_scale), learned
+        self.norm_1, self.mixer, self.norm_2, self.feed_forward = norm_1, mixer, norm_2, feed_forward
+        self.connections = {}          # sublayer -> (in, residual_scale * out, mix)
+
+    def children(self):
+        return tuple(p for p in (self.norm_1, self.mixer, self.norm_2, self.feed_forward) if p is not None)
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def _sublayers(self):
+        return (1,) if self.feed_forward is None else (1, 2)
+
+    def param_specs(self):
+        S, specs = self.n_streams, []
+        if self.learned:
+            for q in self._sublayers():
+                n = f"{self.name}.hc{q}"
+                specs += [ParamSpec(n + ".in", (S,), VECTOR, Init(1.0 / S, 0.3 / S)), ParamSpec(n + ".out", (S,), VECTOR, Init(1.0, 0.2)),
+                          ParamSpec(n + ".mix", (S, S), VECTOR, Init(1.0 / S, 0.3 / S))]
+        return specs
+
+    def bind(self, tensors, dtype, device) -> None:
+        for q in self._sublayers():
+            if self.learned:
+                n = f"{self.name}.hc{q}"
+                w_in, w_out, mix = (tensors[f"{n}.{t}"].contiguous() for t in ("in", "out", "mix"))
+            else:
+                w_in, w_out, mix = (torch.ones(s, dtype=torch.float32, device=device) for s in ((1,), (1,), (1, 1)))
+            self.connections[q] = (w_in, w_out * self.residual_scale, mix)
+
+    def _reader(self, q: int):
+        norm = self.norm_1 if q == 1 else self.norm_2
+        weight, eps = norm.rms_args()
+        return norm, self.connections[q][0], weight, eps
+
+    def _read(self, ctx, x):
+        norm, w_in, weight, eps = self._reader(1)
+        T, D = x.shape[0], norm.width
+        out = ctx.ws.get("normed", T, D, ctx.dtype)
+        ops.label(norm.name, (2.0 * self.n_streams + 4.0) * T * D, (4.0 * self.n_streams + out.element_size()) * T * D)
+        ops.streams_read(x, self.n_streams, w_in, weight, out, eps, ctx.stream)
+        return out
+
+    def _update(self, ctx, x, y, q: int, reader, tag: str):
+        T, D, S = y.shape[0], y.shape[1], self.n_streams
+        _, w_out, mix = self.connections[q]
+        out, kw = None, {}
+        if reader is not None:
+            _, w_in, weight, eps = reader
+            out = ctx.ws.get(tag, T, D, ctx.dtype)
+            kw = dict(nxt=(w_in, weight), next_out=out, eps=eps)
+        ops.label(f"{self.name}.hc{q}", (2.0 * S * S + 4.0 * S + 4.0) * T * D,
+                  (8.0 * S + 4.0 + (out.element_size() if out is not None else 0)) * T * D)
+        ops.streams_update(x, y, S, mix, w_out, ctx.stream, token_req=ctx.token_req, **kw)
+        return out
+
+    def forward(self, ctx, x, cache):
+        carried, ctx.carried = getattr(ctx, "carried", None), None
+        n1 = carried[1] if carried is not None and carried[0] is self else self._read(ctx, x)
+        nxt = getattr(ctx, "next_block", None)
+        if not (isinstance(nxt, HyperBlock) and nxt.n_streams == self.n_streams):
+            nxt = None
+        y = self.mixer.mix(ctx, n1, cache)
+        if self.feed_forward is not None:
+            n2 = self._update(ctx, x, y, 1, self._reader(2), "normed_2")
+            y, terms = self.feed_forward.branch(ctx, n2)
+            if terms != 1:
+                raise ops.KernelError(f"{self.name}: a feed-forward that leaves {terms} rows a token")
+        out = self._update(ctx, x, y, 2 if self.feed_forward is not None else 1, nxt._reader(1) if nxt is not None else None,
+                           "normed")
+        if out is not None:
+            ctx.carried = (nxt, out)
+        return x
+
+
+register_part("block", "hyper", HyperBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "sandwich", SandwichBlock)

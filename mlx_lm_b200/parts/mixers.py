@@ -440,14 +440,20 @@ class LatentAttention(Mixer):
     up-projection is applied to its output (again a product per head), then ``<name>.o``.  Queries and the
     attention's output stay float32 between those products.  Rotation pairs ``(2i, 2i+1)`` (``interleaved``) or
     ``(i, i + rot_dim/2)``, optionally stretched (``rot_scaling``, see ``parts.rotation_frequencies``; the scores' scale
-    stays as given); ``window`` as in the other attention parts."""
+    stays as given); ``window`` as in the other attention parts.
+
+    ``q_rank``: queries go through a latent of their own, ``<name>.uq`` applied to ``<name>.dq x`` RMS-normed with the weight
+    ``<name>.dq.norm`` (instead of ``<name>.q``).  ``head_gate``: head ``h``'s output times ``sigmoid(W_g x)_h`` (``<name>.g``
+    ``[heads, width]``), applied to the head's latent result (the values' up-projection is linear).  ``mix`` returns the
+    output projection in float32 for a block that adds it to the stream itself; ``forward`` adds it in that product's
+    epilogue."""
     replayable = True
     kernel_libs = ("attention_wide", "attention_wide_tc", "latent")
 
     def __init__(self, name: str, width: int, n_heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int,
                  scale: float, eps: float, rot_base: float = 10000.0, interleaved: bool = True,
                  window: Optional[int] = None, chunk: Optional[int] = None, init: Init = Init(),
-                 rot_scaling: Optional[dict] = None):
+                 rot_scaling: Optional[dict] = None, q_rank: Optional[int] = None, head_gate: bool = False):
         if rot_dim % 2:
             raise ValueError(f"{name}: {rot_dim} rotated dimensions")
         self.rot_scaling, self.rot_mscale = rot_scaling, 1.0
@@ -458,14 +464,23 @@ class LatentAttention(Mixer):
         self.q_head = dim + rot_dim
         self.lat = kv_rank + rot_dim                      # what a score is taken over
         self.row = (self.lat + 7) // 8 * 8                # a page row: whole 16 bytes
-        self.proj = FusedLinear(f"{name}.q_dkv", width, [(f"{name}.q", n_heads * self.q_head),
-                                                         (f"{name}.dkv", kv_rank + rot_dim)], init=init)
+        self.q_rank, self.head_gate = q_rank, head_gate
+        sources = [(f"{name}.q", n_heads * self.q_head) if q_rank is None else (f"{name}.dq", int(q_rank)),
+                   (f"{name}.dkv", kv_rank + rot_dim)]
+        if head_gate:
+            sources.append((f"{name}.g", n_heads))
+        self.proj = FusedLinear(f"{name}.q_dkv", width, sources, init=init)
+        self.up_q = None
+        if q_rank is not None:
+            self.up_q = Linear(f"{name}.uq", int(q_rank), n_heads * self.q_head, bias=False, weight_suffix="",
+                               init=Init(0.0, int(q_rank) ** -0.5))
+            self.kernel_libs = type(self).kernel_libs + ("rms",)
         self.out = Linear(f"{name}.o", n_heads * vdim, width, bias=False, weight_suffix="", init=init)
         self.init = init
-        self.norm_w = self.w_absorb = self.w_values = self.freq = None
+        self.norm_w = self.q_norm_w = self.w_absorb = self.w_values = self.freq = None
 
     def children(self):
-        return (self.proj, self.out)
+        return tuple(p for p in (self.proj, self.up_q, self.out) if p is not None)
 
     def cache_spec(self):
         return PagedKVSpec(1, self.row, self.window, chunk=self.chunk, value_dim=0)
@@ -473,13 +488,17 @@ class LatentAttention(Mixer):
     def param_specs(self) -> List[ParamSpec]:
         n, H, R = self.name, self.n_heads, self.rank
         up = Init(0.0, R ** -0.5)
-        return [ParamSpec(f"{n}.dkv.norm", (R,), VECTOR, Init(1.0, 0.1)),
-                ParamSpec(f"{n}.uk", (H * self.dim, R), MATRIX, up),
-                ParamSpec(f"{n}.uv", (H * self.vdim, R), MATRIX, up)]
+        specs = [ParamSpec(f"{n}.dkv.norm", (R,), VECTOR, Init(1.0, 0.1)),
+                 ParamSpec(f"{n}.uk", (H * self.dim, R), MATRIX, up),
+                 ParamSpec(f"{n}.uv", (H * self.vdim, R), MATRIX, up)]
+        if self.q_rank is not None:
+            specs.append(ParamSpec(f"{n}.dq.norm", (self.q_rank,), VECTOR, Init(1.0, 0.1)))
+        return specs
 
     def bind(self, tensors, dtype, device) -> None:
         n, H, R = self.name, self.n_heads, self.rank
         self.norm_w = tensors[f"{n}.dkv.norm"]
+        self.q_norm_w = tensors[f"{n}.dq.norm"] if self.q_rank is not None else None
         # [H, rank, dim]: head h's matrix from its unrotated query to the latent columns
         self.w_absorb = tensors[f"{n}.uk"].view(H, self.dim, R).transpose(1, 2).contiguous()
         self.w_values = tensors[f"{n}.uv"].view(H, self.vdim, R).contiguous()
@@ -488,30 +507,50 @@ class LatentAttention(Mixer):
             self.freq = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(device)
 
     def forward(self, ctx, x, residual, cache):
+        return self.out.forward(ctx, self._heads_out(ctx, x, cache), residual, residual=residual)
+
+    def mix(self, ctx, x, cache, tag: str = "mix_out"):
+        o = self._heads_out(ctx, x, cache)
+        return self.out.forward(ctx, o, ctx.ws.get(tag, x.shape[0], self.width, torch.float32))
+
+    def _heads_out(self, ctx, x, cache):
         T, H, R = x.shape[0], self.n_heads, self.rank
         n = self.proj.n_out
         proj = ctx.ws.get("latent_proj", T, (n + 7) // 8 * 8, x.dtype)[:, :n]
         self.proj.forward(ctx, x, proj)
+        q, c_off = proj[:, :H * self.q_head], self.proj.offset(f"{self.name}.dkv")
+        if self.q_rank is not None:
+            L, HQ = self.q_rank, H * self.q_head
+            cq = ctx.ws.get("latent_cq", T, (L + 7) // 8 * 8, x.dtype)[:, :L]
+            ops.label(self.name + ".dq.norm", 4.0 * T * L, 2.0 * x.element_size() * T * L)
+            ops.rmsnorm(proj[:, :L], self.q_norm_w, cq, self.eps, ctx.stream)
+            q = ctx.ws.get("latent_uq", T, (HQ + 7) // 8 * 8, x.dtype)[:, :HQ]
+            self.up_q.forward(ctx, cq, q)
         q_lat = ctx.ws.get("latent_q", T, H * self.lat, torch.float32)
-        ops.label(self.name + ".prepare", 8.0 * T * n, x.element_size() * T * (n + self.row) + 4.0 * T * H * self.rot_dim)
-        ops.latent_prepare(proj, 0, H * self.q_head, H, self.dim, self.rot_dim, R, self.norm_w, self.eps, self.freq,
+        ops.label(self.name + ".prepare", 8.0 * T * (self.lat + H * self.rot_dim),
+                  x.element_size() * T * (self.lat + H * self.rot_dim + self.row) + 4.0 * T * H * self.rot_dim)
+        ops.latent_prepare(proj, 0, c_off, H, self.dim, self.rot_dim, R, self.norm_w, self.eps, self.freq,
                            self.interleaved, ctx.positions, ctx.token_req, cache.block_table, cache.k, cache.write, q_lat,
-                           self.lat, ctx.status, ctx.stream, mscale=self.rot_mscale)
+                           self.lat, ctx.status, ctx.stream, mscale=self.rot_mscale, queries=q)
         ops.label(self.name + ".uk", 2.0 * T * H * self.dim * R, x.element_size() * (T * H * self.dim + H * self.dim * R)
                   + 4.0 * T * H * R)
-        ops.head_linear(proj, self.q_head, self.w_absorb, q_lat, self.lat, ctx.stream, token_req=ctx.token_req)
+        ops.head_linear(q, self.q_head, self.w_absorb, q_lat, self.lat, ctx.stream, token_req=ctx.token_req)
         o_lat = ctx.ws.get("latent_o", T, H * R, torch.float32)
         if ops.recording():
             pairs, keys = visible_pairs(ctx, self.window, self.chunk)
             ops.label(self.name + ".latent.attention", pairs * H * 2.0 * (self.lat + R),
                       x.element_size() * keys * self.row + 4.0 * T * H * (self.lat + R))
+        gate = None
+        if self.head_gate:
+            g_off = self.proj.offset(f"{self.name}.g")
+            gate = proj[:, g_off:g_off + H]
         ops.attention_wide_step(ctx, q_lat, self.lat, cache.k, cache.k, cache.block_table, o_lat, R, H, self.lat, R,
-                                self.scale, window=self.window or 0, chunk=self.chunk or 0)
+                                self.scale, window=self.window or 0, chunk=self.chunk or 0, gate=gate)
         o = ctx.ws.get("attn_out", T, H * self.vdim, x.dtype)
         ops.label(self.name + ".uv", 2.0 * T * H * self.vdim * R, 4.0 * T * H * R + x.element_size() * (H * self.vdim * R
                   + T * H * self.vdim))
         ops.head_linear(o_lat, R, self.w_values, o, self.vdim, ctx.stream, token_req=ctx.token_req)
-        return self.out.forward(ctx, o, residual, residual=residual)
+        return o
 
 
 class DifferentialAttention(Mixer):

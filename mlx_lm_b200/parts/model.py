@@ -17,8 +17,11 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from .. import ops
-from .base import MATRIX, Block, Init, Norm, ParamSpec, Part, PositionEncoding
+from .base import MATRIX, VECTOR, Block, Init, Norm, ParamSpec, Part, PositionEncoding, StateSpec
 from .linear import Linear
+
+
+EMBEDDING_CACHE = -1    # number of the cache an embedding with state of its own uses (blocks' caches count from 0)
 
 
 @dataclass(frozen=True)
@@ -66,6 +69,50 @@ class TokenEmbedding(Part):
         freq = position.embedding_frequencies() if position is not None else None
         ops.embed_pos(ctx.tokens, ctx.positions, self.table, table, x, ctx.status, ctx.stream, scale=self.scale,
                       freq=freq)
+        return x
+
+
+class TokenPairEmbedding(Part):
+    """``norm(table[token] * scale + pairs[row])``, written once for each of ``n_streams`` streams of a float32 residual
+    (``[T, n_streams * width]``).  ``row = (token before * mul_prev + token * mul_cur) mod buckets``; a sequence's first token
+    takes the last row of ``pairs`` (``[buckets + 1, width]``).  The token before is part of a request's state (one number
+    in its slot: ``cache_spec()``).  ``buckets=0``: no table of pairs and no state.  The norm is an RMS norm over the width
+    with the weight ``norm_name``."""
+    replayable = True
+    kernel_libs = ("embed",)
+
+    def __init__(self, name: str, vocab_size: int, width: int, eps: float, scale: float = 1.0, pairs_name: str = "bigram",
+                 buckets: int = 0, mul_prev: int = 0, mul_cur: int = 0, norm_name: str = "embed.norm", n_streams: int = 1,
+                 init: Init = Init(), weight_suffix: str = ""):
+        if vocab_size > 1 << 24:
+            raise ValueError(f"{name}: the state keeps token ids in float32, which holds them exactly up to {1 << 24}")
+        self.name, self.vocab_size, self.width, self.eps, self.scale, self.init = name, vocab_size, width, float(eps), float(scale), init
+        self.weight_name, self.norm_name = name + weight_suffix, norm_name
+        self.pairs_name, self.buckets, self.mul_prev, self.mul_cur = pairs_name, int(buckets), int(mul_prev), int(mul_cur)
+        self.n_streams = int(n_streams)
+        self.table = self.pairs = self.norm_w = None
+
+    def cache_spec(self):
+        return StateSpec((1,)) if self.buckets else None
+
+    def param_specs(self) -> List[ParamSpec]:
+        specs = [ParamSpec(self.weight_name, (self.vocab_size, self.width), MATRIX, self.init)]
+        if self.buckets:
+            specs.append(ParamSpec(self.pairs_name, (self.buckets + 1, self.width), MATRIX,
+                                   Init(0.0, self.init.std * self.scale)))
+        return specs + [ParamSpec(self.norm_name, (self.width,), VECTOR, Init(1.0, 0.1))]
+
+    def bind(self, tensors, dtype, device) -> None:
+        self.table, self.norm_w = tensors[self.weight_name], tensors[self.norm_name]
+        self.pairs = tensors[self.pairs_name] if self.buckets else None
+
+    def forward(self, ctx, position: Optional[PositionEncoding], cache=None):
+        T, D, S = ctx.n_tokens, self.width, self.n_streams
+        x = ctx.ws.get("residual", T, S * D, torch.float32)
+        ops.label(self.name, 6.0 * T * D, ((2 if self.buckets else 1) * self.table.element_size() + 4.0 * S) * T * D)
+        ops.embed_pairs(ctx.tokens, ctx.positions, ctx.token_req, ctx.req_first_token, ctx._slots, self.table, self.pairs,
+                        cache.state if self.buckets else None, self.norm_w, x, S, ctx.status, ctx.stream, scale=self.scale,
+                        buckets=self.buckets, mul_prev=self.mul_prev, mul_cur=self.mul_cur, eps=self.eps)
         return x
 
 
@@ -174,9 +221,12 @@ class ModelDescription:
         return list(dict.fromkeys(libs))
 
     def cache_specs(self) -> Dict[object, object]:
-        """Every cache the run order uses.  A block with one cache: ``cache number -> spec``; a block whose
+        """Every cache the run order uses, and the embedding's (``EMBEDDING_CACHE``) where it keeps state.  A block with one cache: ``cache number -> spec``; a block whose
         ``cache_spec()`` is a dictionary (several caches under names): ``(cache number, name) -> spec``."""
         out = {}
+        embedding = self.embedding.cache_spec() if hasattr(self.embedding, "cache_spec") else None
+        if embedding is not None:
+            out[EMBEDDING_CACHE] = embedding
         for c, b in self.cache_owner().items():
             spec = self.blocks[b].cache_spec()
             if isinstance(spec, dict):
@@ -223,13 +273,19 @@ class Model:
         """All of this step's tokens through the blocks in run order; float32 logits
         ``[len(ctx.logit_rows), vocab]`` at the wanted rows, or None if none is wanted."""
         d = self.description
-        x = x0 = d.embedding.forward(ctx, d.position)
+        if getattr(d.embedding, "cache_spec", None) is not None:
+            x = x0 = d.embedding.forward(ctx, d.position, ctx.cache_view(RunEntry(0, cache=EMBEDDING_CACHE)))
+        else:
+            x = x0 = d.embedding.forward(ctx, d.position)
         if d.reentries and not isinstance(d.order[0], Reentry):
             # blocks that run before the first reentry change the stream in place: they get a copy, the embedding
             # output stays as it is for the reentries
             x = ctx.ws.get("stream", ctx.n_tokens, d.width, x0.dtype)
             ops.join_rows(x0, None, x, ctx.stream)
-        for entry in d.order:
+        for i, entry in enumerate(d.order):
+            after = d.order[i + 1] if i + 1 < len(d.order) else None
+            # the block that reads the stream next, for a block that prepares its input in the same pass
+            ctx.next_block = d.blocks[after.block] if isinstance(after, RunEntry) else None
             if isinstance(entry, Reentry):
                 x = d.reentries[entry.part].forward(ctx, x, x0, entry.index)
             else:
@@ -261,7 +317,6 @@ class LoopInput(Part):
         return (self.linear,)
 
     def param_specs(self) -> List[ParamSpec]:
-        from .base import VECTOR
         return [ParamSpec(self.step_name, (self.times, self.width), VECTOR, Init(0.0, 0.1))]
 
     def bind(self, tensors, dtype, device) -> None:

@@ -6,6 +6,8 @@ from __future__ import annotations
 
 from typing import List, Optional
 
+import torch
+
 from .. import ops
 from .base import VECTOR, Init, Norm, ParamSpec, register_part
 
@@ -52,19 +54,49 @@ class RMSNorm(Norm):
         self.name, self.width, self.eps, self.offset = name, width, float(eps), float(offset)
         self.weight_name = name + weight_suffix
         self.init = init if init is not None else Init(1.0 - self.offset, 0.1)
-        self.weight = None
+        self.weight = self._plain = None
 
     def param_specs(self) -> List[ParamSpec]:
         return [ParamSpec(self.weight_name, (self.width,), VECTOR, self.init)]
 
     def bind(self, tensors, dtype, device) -> None:
-        self.weight = tensors[self.weight_name]
+        self.weight, self._plain = tensors[self.weight_name], None
 
     def forward(self, ctx, x, rows=None, tag: str = "normed"):
         n = x.shape[0] if rows is None else rows.numel()
         out = ctx.ws.get(tag, n, self.width, ctx.dtype)
         ops.label(self.name, 4.0 * n * self.width, (4.0 + out.element_size()) * n * self.width)
         ops.rmsnorm(x, self.weight, out, self.eps, ctx.stream, offset=self.offset, rows=rows)
+        return out
+
+    def rms_args(self):
+        """``(weight, eps)`` of the norm written with a plain weight, for a kernel that applies it in passing."""
+        if self._plain is None:
+            self._plain = self.weight if self.offset == 0.0 else self.weight + self.offset
+        return self._plain, self.eps
+
+
+class StreamsNorm(RMSNorm):
+    """The RMS norm of the sum of ``n_streams`` residual streams (rows ``[x_1 | .. | x_S]``): what a model with several
+    streams puts before its output head."""
+    kernel_libs = ("streams",)
+
+    def __init__(self, name: str, width: int, eps: float, n_streams: int, offset: float = 0.0, weight_suffix: str = "",
+                 init: Optional[Init] = None):
+        super().__init__(name, width, eps, offset, weight_suffix, init)
+        self.n_streams = int(n_streams)
+        self.ones = None
+
+    def bind(self, tensors, dtype, device) -> None:
+        super().bind(tensors, dtype, device)
+        self.ones = torch.ones(self.n_streams, dtype=torch.float32, device=device)
+
+    def forward(self, ctx, x, rows=None, tag: str = "normed"):
+        n = x.shape[0] if rows is None else rows.numel()
+        out = ctx.ws.get(tag, n, self.width, ctx.dtype)
+        weight, eps = self.rms_args()
+        ops.label(self.name, (self.n_streams + 4.0) * n * self.width, (4.0 * self.n_streams + out.element_size()) * n * self.width)
+        ops.streams_read(x, self.n_streams, self.ones, weight, out, eps, ctx.stream, rows=rows)
         return out
 
 
@@ -111,3 +143,4 @@ class DynamicTanh(Norm):
 register_part("norm", "layer_norm", LayerNorm)
 register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "rms_norm", RMSNorm)
+register_part("norm", "streams_norm", StreamsNorm)

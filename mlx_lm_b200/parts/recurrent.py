@@ -1,5 +1,6 @@
 """Mixers that keep a state of fixed size per request instead of keys and values: the selective
-state-space layer of Mamba-2 and the gated delta rule.  Both read their inputs through short causal
+state-space layer of Mamba-2, the gated delta rule, RWKV's time mixing, retention and the real-gated linear
+recurrent unit.  Some read their inputs through short causal
 convolutions whose last ``taps - 1`` inputs are part of the state.  State is float32 and lives in the
 cache manager's slots; a step reads it at the start of each request's run of tokens and writes it back
 at the end, so prompts may be cut into portions anywhere and decoding continues from it.
@@ -10,13 +11,14 @@ else); ``forward`` adds it to a float32 residual stream in that projection's epi
 
 from __future__ import annotations
 
-from typing import List
+from typing import List, Sequence
 
 import torch
 
 from .. import ops
-from .base import VECTOR, Init, Mixer, ParamSpec, StateSpec, register_part
+from .base import MATRIX, VECTOR, Init, Mixer, ParamSpec, StateSpec, register_part
 from .linear import FusedLinear, Linear
+from .positions import rotation_frequencies
 
 
 class Mamba2Mixer(Mixer):
@@ -254,6 +256,148 @@ class WKVMixer(Mixer):
         return self.out.forward(ctx, self._gated(ctx, x, cache), residual, residual=residual)
 
 
+class RetentionMixer(Mixer):
+    """Linear attention with a fixed decay per head, without softmax or denominator.  ``q``, ``k`` (``heads x dim``), ``v``
+    (``heads x vdim``); the first ``rot_dims`` dimensions of every q and k head turn with the position (pairs
+    ``(i, i + rot_dims/2)``, angle ``p * rot_base**(-2i/rot_dims)``), k times ``dim**-0.5`` after that; per head
+    ``S <- decay_h S + k v^T``, ``o = S^T q``; every head's ``o`` is divided by its root mean square (eps inside the root, no
+    weight), times ``silu(g x)``, then ``o``.  Everything between the projections and the gate is float32."""
+    replayable = True
+    kernel_libs = ("retention", "rms")
+
+    def __init__(self, name: str, width: int, n_heads: int, dim: int, vdim: int, decay: Sequence[float], eps: float,
+                 rot_dims: int = 0, rot_base: float = 10000.0, init: Init = Init()):
+        if len(decay) != n_heads:
+            raise ValueError(f"{name}: {len(decay)} decays for {n_heads} heads")
+        if rot_dims % 2 or rot_dims > dim:
+            raise ValueError(f"{name}: {rot_dims} rotated dimensions of {dim}")
+        self.name, self.width, self.n_heads, self.dim, self.vdim = name, width, n_heads, dim, vdim
+        self.decay_list, self.eps = [float(d) for d in decay], float(eps)
+        self.rot_dims, self.rot_base = rot_dims, float(rot_base)
+        self.qk_width, self.v_width = n_heads * dim, n_heads * vdim
+        self.proj = FusedLinear(f"{name}.qkvg", width, [(f"{name}.q", self.qk_width), (f"{name}.k", self.qk_width),
+                                                        (f"{name}.v", self.v_width), (f"{name}.g", self.v_width)], init=init)
+        self.out = Linear(f"{name}.o", self.v_width, width, bias=False, weight_suffix="", init=Init(0.0, self.v_width ** -0.5))
+        self.decay = self.freq = None
+
+    def children(self):
+        return (self.proj, self.out)
+
+    def cache_spec(self):
+        return StateSpec((self.n_heads, self.vdim, self.dim))      # column by column: the scan's layout
+
+    def bind(self, tensors, dtype, device) -> None:
+        self.decay = torch.tensor(self.decay_list, dtype=torch.float32, device=device)
+        if self.rot_dims:
+            f, _ = rotation_frequencies(self.rot_dims, self.rot_base)
+            self.freq = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(device)
+
+    def _gated(self, ctx, x, cache):
+        T, H, VW = x.shape[0], self.n_heads, self.v_width
+        n = self.proj.n_out
+        proj = ctx.ws.get("retention_proj", T, (n + 7) // 8 * 8, x.dtype)[:, :n]
+        self.proj.forward(ctx, x, proj)
+        v_off = 2 * self.qk_width
+        o = ctx.ws.get("retention_o", T, VW, torch.float32)
+        ops.label(self.name + ".scan", 6.0 * T * VW * self.dim, x.element_size() * T * (v_off + VW) + 4.0 * T * VW
+                  + 8.0 * min(T, ctx.n_requests) * VW * self.dim)
+        ops.retention_scan(proj, 0, self.qk_width, v_off, self.freq, self.dim ** -0.5, self.decay, cache.state, cache.slots,
+                           ctx.positions, ctx.token_req, ctx.req_first_token, o, H, ctx.stream)
+        g = ctx.ws.get("retention_gated", T, VW, x.dtype)
+        ops.label(self.name + ".norm", 8.0 * T * VW, (4.0 + 2 * x.element_size()) * T * VW)
+        ops.rmsnorm(o, None, g, self.eps, ctx.stream, groups=H, gate=proj[:, v_off + VW:v_off + 2 * VW],
+                    gate_mode=ops.GATE_AFTER)
+        return g
+
+    def mix(self, ctx, x, cache, tag: str = "mix_out"):
+        g = self._gated(ctx, x, cache)
+        return self.out.forward(ctx, g, ctx.ws.get(tag, x.shape[0], self.width, torch.float32))
+
+    def forward(self, ctx, x, residual, cache):
+        return self.out.forward(ctx, self._gated(ctx, x, cache), residual, residual=residual)
+
+
+class RGLRUMixer(Mixer):
+    """A recurrent block of two branches of ``inner`` columns: ``y = gelu_tanh(W_y x + b)`` and ``u``, a short causal
+    convolution with bias (``<name>.conv`` ``[inner, taps]``, ``<name>.conv.b``; no activation) of ``W_x x + b``, through a
+    real-gated linear recurrent unit.  ``u`` is cut into ``blocks`` equal parts with square matrices of their own:
+    ``r = sigmoid(ra_b u_b + ra.b_b)``, ``i = sigmoid(ri_b u_b + ri.b_b)``; per channel ``log a = -8 r softplus(lam)``,
+    ``S <- a S + sqrt(1 - a^2) i u``; ``<name>.o`` of ``S * y``.  Gates, decays and the state are float32 (the gates'
+    products: float32 sums, left in float32)."""
+    replayable = True
+    kernel_libs = ("recurrent", "rglru", "latent")
+
+    def __init__(self, name: str, width: int, inner: int, blocks: int, taps: int, init: Init = Init()):
+        if blocks < 1 or inner % blocks:
+            raise ValueError(f"{name}: {inner} channels in {blocks} equal parts")
+        if not 1 <= taps <= 9:
+            raise ValueError(f"{name}: a convolution of {taps} taps (1 to 9)")
+        self.name, self.width, self.inner, self.blocks, self.taps = name, width, inner, blocks, taps
+        self.block = inner // blocks
+        self.inner_p = (inner + 7) // 8 * 8
+        self.proj = FusedLinear(f"{name}.yx", width, [(f"{name}.y", inner), (f"{name}.x", inner)], init=init,
+                                biases={f"{name}.y": f"{name}.y.b", f"{name}.x": f"{name}.x.b"}, bias_init=Init(0.0, 0.1))
+        self.out = Linear(f"{name}.o", inner, width, bias=False, weight_suffix="", init=Init(0.0, inner ** -0.5))
+        self._no_state = None
+
+    def children(self):
+        return (self.proj, self.out)
+
+    def cache_spec(self):
+        spec = {"unit": StateSpec((self.inner,))}
+        if self.taps > 1:
+            spec["conv"] = StateSpec((self.taps - 1, self.inner))
+        return spec
+
+    def param_specs(self) -> List[ParamSpec]:
+        n, W, B, b = self.name, self.inner, self.blocks, self.block
+        gate = Init(0.0, b ** -0.5)
+        return [ParamSpec(f"{n}.conv", (W, self.taps), VECTOR, Init(0.0, 0.4)), ParamSpec(f"{n}.conv.b", (W,), VECTOR, Init(0.0, 0.1)),
+                ParamSpec(f"{n}.ra", (B, b, b), MATRIX, gate), ParamSpec(f"{n}.ra.b", (B, b), VECTOR, Init(0.0, 0.1)),
+                ParamSpec(f"{n}.ri", (B, b, b), MATRIX, gate), ParamSpec(f"{n}.ri.b", (B, b), VECTOR, Init(0.0, 0.1)),
+                ParamSpec(f"{n}.lam", (W,), VECTOR, Init(-4.0, 1.0))]
+
+    def bind(self, tensors, dtype, device) -> None:
+        n = self.name
+        self.conv_w, self.conv_b = tensors[f"{n}.conv"].contiguous(), tensors[f"{n}.conv.b"].contiguous()
+        self.conv_wt = self.conv_w.t().contiguous()
+        # [blocks, 2 * block, block]: a part's recurrence gate, then its input gate, as one product per part
+        self.w_gates = torch.cat([tensors[f"{n}.ra"], tensors[f"{n}.ri"]], dim=1).contiguous()
+        self.r_bias, self.i_bias = (tensors[f"{n}.{t}.b"].reshape(-1).contiguous() for t in ("ra", "ri"))
+        lam = tensors[f"{n}.lam"].double()
+        self.decay = (-8.0 * torch.logaddexp(lam, torch.zeros_like(lam))).float().contiguous()
+        self._no_state = torch.zeros((1, 0, self.inner), dtype=torch.float32, device=device)
+
+    def _gated(self, ctx, x, cache):
+        T, W, es = x.shape[0], self.inner, x.element_size()
+        yx = ctx.ws.get("rglru_yx", T, 2 * self.inner_p, x.dtype)[:, :2 * W]
+        self.proj.forward(ctx, x, yx)
+        y, xb = yx[:, :W], yx[:, W:]
+        u = ctx.ws.get("rglru_u", T, self.inner_p, x.dtype)[:, :W]
+        state, slots = (cache.side("conv").state, cache.side("conv").slots) if self.taps > 1 else (self._no_state, ctx._slots)
+        ops.label(self.name + ".conv", 2.0 * self.taps * T * W, 2.0 * es * T * W)
+        ops.conv_silu(xb, self.conv_w, self.conv_b, state, slots, ctx.positions, ctx.token_req, ctx.req_first_token,
+                      ctx.req_first_position, u, ctx.stream, weight_by_tap=self.conv_wt, activation=False)
+        gates = ctx.ws.get("rglru_gates", T, 2 * W, torch.float32)
+        ops.label(self.name + ".gates", 4.0 * T * W * self.block, es * (T * W + 2 * W * self.block) + 8.0 * T * W)
+        ops.head_linear(u, self.block, self.w_gates, gates, 2 * self.block, ctx.stream, token_req=ctx.token_req)
+        unit = cache.side("unit")
+        out = ctx.ws.get("rglru_out", T, self.inner_p, x.dtype)[:, :W]
+        ops.label(self.name + ".scan", 30.0 * T * W, (8.0 + 3 * es) * T * W + 8.0 * min(T, ctx.n_requests) * W)
+        ops.rglru_scan(gates, self.r_bias, self.i_bias, self.decay, u, y, unit.state, unit.slots, ctx.token_req,
+                       ctx.req_first_token, out, self.block, ctx.stream, singles=ctx.n_single > 0, portions=ctx.n_portion > 0)
+        return out
+
+    def mix(self, ctx, x, cache, tag: str = "mix_out"):
+        g = self._gated(ctx, x, cache)
+        return self.out.forward(ctx, g, ctx.ws.get(tag, x.shape[0], self.width, torch.float32))
+
+    def forward(self, ctx, x, residual, cache):
+        return self.out.forward(ctx, self._gated(ctx, x, cache), residual, residual=residual)
+
+
+register_part("mixer", "retention", RetentionMixer)
+register_part("mixer", "rglru", RGLRUMixer)
 register_part("mixer", "mamba2", Mamba2Mixer)
 register_part("mixer", "wkv", WKVMixer)
 register_part("mixer", "gated_delta", GatedDeltaMixer)
