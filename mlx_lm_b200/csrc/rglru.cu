@@ -5,6 +5,10 @@
 //   S_t = exp(log a) S_(t-1) + sqrt(1 - exp(2 log a)) * i * u_t
 //   out_t = S_t * gelu_tanh(y_t)                        rounded once to the activation dtype
 //
+// The decay is formed as 1 + x and the factor as sqrt(-x (2 + x)) with x = exp(log a) - 1 (expm1f): both keep their
+// accuracy where a is close to one.  (A channel that forgets slowly multiplies by nearly the same a for a thousand rows: the
+// error of a float32 exponential, a unit or two in the last place, adds up; that of 1 + x is half a unit at most.)
+//
 // S is float32, one number per channel and request ([slots, W]), read at the start of the run of rows a step brings for
 // the request (req_first_token[r] .., as many as carry its index in token_req) and written back at its end.
 //
@@ -82,8 +86,9 @@ rglru_scan_kernel(const float* gates, int ldg, const float* __restrict__ br, con
     for (int e = 0; e < RG_LEN; ++e) {
       const bool in = lo + e < n;
       const float la = sigmoid_f(pr[e] + b_r) * cd;
-      a[e] = in ? expf(la) : 1.f;
-      b[e] = in ? sqrtf(-expm1f(2.f * la)) * (sigmoid_f(pi[e] + b_i) * uu[e]) : 0.f;
+      const float x = expm1f(la);
+      a[e] = in ? 1.f + x : 1.f;
+      b[e] = in ? sqrtf(-x * (2.f + x)) * (sigmoid_f(pi[e] + b_i) * uu[e]) : 0.f;
       A *= a[e];
       B = fmaf(a[e], B, b[e]);
     }
@@ -131,7 +136,8 @@ __global__ void rglru_row_kernel(const float* gates, int ldg, const float* __res
   const float* gp = gates + (size_t)t0 * ldg + (size_t)blk * 2 * n_block + j;
   const float pr = gp[0], pi = gp[n_block], uu = to_f(u[(size_t)t0 * ldu + c]), yy = to_f(y[(size_t)t0 * ldy + c]);
   const float la = sigmoid_f(pr + b_r) * cd;
-  const float S = fmaf(expf(la), S0, sqrtf(-expm1f(2.f * la)) * (sigmoid_f(pi + b_i) * uu));
+  const float x = expm1f(la);
+  const float S = fmaf(1.f + x, S0, sqrtf(-x * (2.f + x)) * (sigmoid_f(pi + b_i) * uu));
   *sp = S;
   out[(size_t)t0 * ldo + c] = from_f<T>(S * gelu_y<T>(yy));
 }
