@@ -731,6 +731,38 @@ def zuluvik_config(width, vocab):
             "layers": layers}
 
 
+def vobusun_config(width, vocab):
+    """Ten layer runs of the sizes a model of this width would have, four residual streams: latent rows of 256 + 32
+    columns in a window of 1024 with queries through a latent of half the width; retention with heads of 64 x 128; recurrent
+    blocks of the model's width in parts of 128 behind convolutions of four taps; a feed-forward of about 2.7 times the
+    width on every layer; pairs of tokens in a table of 4093 rows.  Two layers run earlier layers' weights again."""
+    H = width // 64
+    ff = {"ff": (width * 11 // 4 + 127) // 128 * 128, "kind": "dense", "limit": 7.0}
+    lat = {"type": "latent_attention", "mlp": ff,
+           "mixer": {"dim": 64, "heads": H, "kv_rank": 256, "q_rank": width // 2, "rot_dim": 32, "vdim": 64, "scale": 0.1,
+                     "mask": {"size": 1024}, "rot": {"base": 500000.0, "dims": 32}}}
+    ret = {"type": "retention", "mlp": ff,
+           "mixer": {"dim": 64, "heads": H // 2, "vdim": 128, "decay": [1.0 - 2.0 ** -(5 + 3 * h / (H // 2)) for h in range(H // 2)],
+                     "rot": {"base": 10000.0, "dims": 64}}}
+    rec = {"type": "rglru", "mlp": ff, "mixer": {"width": width, "blocks": width // 128, "conv": 4}}
+    layers = [lat, rec, ret, ret, rec, lat, ret, rec, dict(lat, weights_of=0), dict(ret, weights_of=2)]
+    return {"architecture": "Vobusun", "vocab": vocab, "width": width, "streams": 4, "residual_mult": 0.7, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 8.0, "bigram": {"buckets": 4093, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
+
+
+def run_vobusun(args):
+    """The same measurements as ``--only zuluvik`` for the Vobusun design, beside Nufetar (the nearest design in the tree: a
+    float32 stream, attention over latent rows in a window, a linear recurrence per head, dense feed-forwards) and Lelatar
+    (short convolutions and scans) at equal width and as many layer runs."""
+    vocab = 32000
+
+    def models(width):
+        vob = vobusun_config(width, vocab)
+        return len(vob["layers"]), [("vobusun", vob), ("nufetar", nufetar_config(width, vocab)),
+                                    ("lelatar", lelatar_config(width, vocab))]
+    run_beside(args, "vobusun_vs_nufetar", models)
+
+
 def run_zuluvik(args):
     """The same measurements as ``--only dalorax`` for the Zuluvik design, beside Dalorax (the nearest design in the
     tree: a float32 stream, grouped-query attention over pages and mixtures of experts) and Nufetar (attention over
@@ -865,9 +897,9 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration's 24 (0 = all)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--widths", default="", help="with --only lelatar / nufetar / dalorax / zuluvik: the model widths to run, with commas (default 1024,2048)")
+    ap.add_argument("--widths", default="", help="with --only lelatar / nufetar / dalorax / zuluvik / vobusun: the model widths to run, with commas (default 1024,2048)")
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "mixed", "timeline", "kernels", "yardstick",
-                                                   "lelatar", "nufetar", "dalorax", "zuluvik"],
+                                                   "lelatar", "nufetar", "dalorax", "zuluvik", "vobusun"],
                     help="run just this part and print its figures (decode / prefill: short runs for profiling; "
                          "mixed: 64 requests with prompts of 16..1024 tokens through the scheduler, 256-token portions "
                          "beside decoding requests; timeline: every kernel of one step with its start and end, "
@@ -876,7 +908,8 @@ def main():
                          "model's linear shapes, to hold the hand-written kernels against; lelatar: prefill and decode of "
                          "the Lelatar design at two widths beside GPT-2 of equal width and layer runs, with every kernel "
                          "of both against its roofline; nufetar: the same for the Nufetar design beside Lelatar; dalorax: the same for the Dalorax design "
-                         "beside Nufetar; zuluvik: the same for the Zuluvik design beside Dalorax and Nufetar)")
+                         "beside Nufetar; zuluvik: the same for the Zuluvik design beside Dalorax and Nufetar; "
+                         "vobusun: the same for the Vobusun design beside Nufetar and Lelatar)")
     ap.add_argument("--prefill-prompts", type=int, default=0,
                     help="with --only prefill: 1024-token prompts in the one step (default and the contract's figure: "
                          "2); with --only timeline: the timeline of such a step instead of a decode step")
@@ -903,6 +936,9 @@ def main():
         return 0
     if a.only == "zuluvik":
         run_zuluvik(a)
+        return 0
+    if a.only == "vobusun":
+        run_vobusun(a)
         return 0
     run_ours(a)
     return 0

@@ -1029,6 +1029,64 @@ def retention_scan(qkv, q_off: int, k_off: int, v_off: int, freq, kscale: float,
           _rows(o, "retention_scan o"), H, K, V, slots.numel(), int(max_run), stream)
 
 
+RETENTION_TILE = 128      # rows of a tile of retention_chunks at most; the table of a decay's powers has one more entry
+
+
+def retention_chunks_supported(dtype, dim: int, tile_rows: int = 0) -> bool:
+    """Whether runs of several rows go through ``retention_chunks`` (bfloat16, heads of up to 256 key columns)."""
+    return dtype == torch.bfloat16 and 1 <= dim <= 256 and (tile_rows or PREFILL_TILE) <= RETENTION_TILE
+
+
+def retention_chunks_scratch(n_tokens: int, n_requests: int, n_heads: int, dim: int, vdim: int, tile_rows: int = 0) -> int:
+    """Floats of scratch memory ``retention_chunks`` needs: a state per tile of a run."""
+    return (n_tokens // (tile_rows or PREFILL_TILE) + n_requests + 1) * n_heads * dim * vdim
+
+
+def retention_chunks(qkv, q_off: int, k_off: int, v_off: int, freq, kscale: float, powers, state, slots, token_req,
+                     req_first_token, req_first_position, tiles, n_tiles: int, scratch, n_heads: int, stream, out=None,
+                     gate=None, gated=None, eps: float = 0.0, tile_rows: int = 0) -> None:
+    """``retention_scan`` for the requests that bring several rows, in tiles on tensor cores (bfloat16; three launches):
+    a tile's contribution to the state, the states along each run, the tiles' outputs.  ``powers``: float32
+    ``[heads, RETENTION_TILE + 1]``, the powers 0, 1, .. of every head's decay; ``tiles``: int32 ``[n_tiles, 4]`` = (first token
+    row, rows, request, first position), at most ``tile_rows`` rows each.  ``out``: float32 ``[T, heads*V]``; or, with ``gate``
+    and ``gated`` (bfloat16 ``[T, heads*V]``, at most 128 value columns a head), every head's row divided by its root mean
+    square (``eps`` inside the root) and multiplied by ``silu(gate)``."""
+    _need(qkv, torch.bfloat16, "retention_chunks qkv")
+    _need(state, torch.float32, "retention_chunks state")
+    _need(powers, torch.float32, "retention_chunks powers")
+    _need(tiles, torch.int32, "retention_chunks tiles")
+    _need(scratch, torch.float32, "retention_chunks scratch")
+    _, H, V, K = state.shape
+    T, tile_rows = qkv.shape[0], tile_rows or PREFILL_TILE
+    if H != n_heads or not state.is_contiguous() or powers.shape != (H, RETENTION_TILE + 1) or not powers.is_contiguous() \
+            or tiles.numel() < 4 * n_tiles \
+            or scratch.numel() < retention_chunks_scratch(T, slots.numel(), H, K, V, tile_rows):
+        raise KernelError(f"retention_chunks: state {tuple(state.shape)} for {n_heads} heads, powers {tuple(powers.shape)}, "
+                          f"{n_tiles} tiles, scratch of {scratch.numel()}")
+    if (gate is None) != (gated is None) or (out is None) == (gate is None):
+        raise KernelError("retention_chunks: either out, or gate and gated")
+    half = 0
+    if freq is not None:
+        _need(freq, torch.float32, "retention_chunks freq")
+        half = freq.numel()
+    if out is not None:
+        _need(out, torch.float32, "retention_chunks out")
+    else:
+        _need(gate, torch.bfloat16, "retention_chunks gate")
+        _need(gated, torch.bfloat16, "retention_chunks gated")
+    for t in (out, gate, gated):
+        if t is not None and t.shape != (T, H * V):
+            raise KernelError(f"retention_chunks: rows of {tuple(t.shape)} for {H} heads of {V}")
+    rows = lambda t: 0 if t is None else _rows(t, "retention_chunks rows")
+    _call("retention", "mlxb_retention_chunks", [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float]
+          + [c_void_p] * 7 + [c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_float]
+          + [c_int] * 4 + [c_void_p],
+          _p(qkv), _rows(qkv, "retention_chunks qkv"), q_off, k_off, v_off, _p(freq), half, float(kscale), _p(powers),
+          _p(state), _p(slots), _p(token_req), _p(req_first_token), _p(req_first_position), _p(tiles), int(n_tiles),
+          int(tile_rows), _p(scratch), _p(out), rows(out), _p(gate), rows(gate), _p(gated), rows(gated), float(eps), H, K, V,
+          slots.numel(), stream)
+
+
 def rglru_scan(gates, r_bias, i_bias, decay, u, y, state, slots, token_req, req_first_token, out, block: int, stream,
                singles: bool = True, portions: bool = True) -> None:
     """Per channel: ``S <- a S + sqrt(1 - a^2) i u`` and ``out = S * gelu_tanh(y)`` with ``r``, ``i`` the sigmoids of the

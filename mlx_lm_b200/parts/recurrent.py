@@ -278,7 +278,7 @@ class RetentionMixer(Mixer):
         self.proj = FusedLinear(f"{name}.qkvg", width, [(f"{name}.q", self.qk_width), (f"{name}.k", self.qk_width),
                                                         (f"{name}.v", self.v_width), (f"{name}.g", self.v_width)], init=init)
         self.out = Linear(f"{name}.o", self.v_width, width, bias=False, weight_suffix="", init=Init(0.0, self.v_width ** -0.5))
-        self.decay = self.freq = None
+        self.decay = self.powers = self.freq = None
 
     def children(self):
         return (self.proj, self.out)
@@ -288,6 +288,9 @@ class RetentionMixer(Mixer):
 
     def bind(self, tensors, dtype, device) -> None:
         self.decay = torch.tensor(self.decay_list, dtype=torch.float32, device=device)
+        # the powers of every head's decay, from its float32 value as the token-by-token form multiplies it
+        n = torch.arange(ops.RETENTION_TILE + 1, dtype=torch.float64)
+        self.powers = (self.decay.double().cpu()[:, None] ** n[None, :]).float().to(device).contiguous()
         if self.rot_dims:
             f, _ = rotation_frequencies(self.rot_dims, self.rot_base)
             self.freq = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(device)
@@ -298,15 +301,28 @@ class RetentionMixer(Mixer):
         proj = ctx.ws.get("retention_proj", T, (n + 7) // 8 * 8, x.dtype)[:, :n]
         self.proj.forward(ctx, x, proj)
         v_off = 2 * self.qk_width
-        o = ctx.ws.get("retention_o", T, VW, torch.float32)
-        ops.label(self.name + ".scan", 6.0 * T * VW * self.dim, x.element_size() * T * (v_off + VW) + 4.0 * T * VW
-                  + 8.0 * min(T, ctx.n_requests) * VW * self.dim)
-        ops.retention_scan(proj, 0, self.qk_width, v_off, self.freq, self.dim ** -0.5, self.decay, cache.state, cache.slots,
-                           ctx.positions, ctx.token_req, ctx.req_first_token, o, H, ctx.stream)
+        gate = proj[:, v_off + VW:v_off + 2 * VW]
         g = ctx.ws.get("retention_gated", T, VW, x.dtype)
+        where = (ctx.token_req, ctx.req_first_token)
+        tiled = (ctx.n_portion > 0 and ctx.portion_tiles is not None and ops.retention_chunks_supported(x.dtype, self.dim))
+        cost = (6.0 * T * VW * self.dim, x.element_size() * T * (v_off + VW) + 8.0 * min(T, ctx.n_requests) * VW * self.dim)
+        fused = tiled and ctx.n_single == 0 and self.vdim <= 128      # the tiles' own kernel norms and gates their rows
+        o = None if fused else ctx.ws.get("retention_o", T, VW, torch.float32)
+        if tiled:
+            scratch = ctx.ws.flat("retention_states", ops.retention_chunks_scratch(T, ctx.n_requests, H, self.dim, self.vdim),
+                                  torch.float32)
+            ops.label(self.name + ".retention", cost[0], cost[1] + (2.0 * x.element_size() if fused else 4.0) * T * VW)
+            ops.retention_chunks(proj, 0, self.qk_width, v_off, self.freq, self.dim ** -0.5, self.powers, cache.state,
+                                 cache.slots, *where, ctx.req_first_position, ctx.portion_tiles, ctx.n_portion_tiles, scratch, H,
+                                 ctx.stream, **(dict(gate=gate, gated=g, eps=self.eps) if fused else dict(out=o)))
+            if fused:
+                return g
+        if not tiled or ctx.n_single:
+            ops.label(self.name + ".retention", cost[0], cost[1] + 4.0 * T * VW)
+            ops.retention_scan(proj, 0, self.qk_width, v_off, self.freq, self.dim ** -0.5, self.decay, cache.state, cache.slots,
+                               ctx.positions, *where, o, H, ctx.stream, max_run=1 if tiled else 0)
         ops.label(self.name + ".norm", 8.0 * T * VW, (4.0 + 2 * x.element_size()) * T * VW)
-        ops.rmsnorm(o, None, g, self.eps, ctx.stream, groups=H, gate=proj[:, v_off + VW:v_off + 2 * VW],
-                    gate_mode=ops.GATE_AFTER)
+        ops.rmsnorm(o, None, g, self.eps, ctx.stream, groups=H, gate=gate, gate_mode=ops.GATE_AFTER)
         return g
 
     def mix(self, ctx, x, cache, tag: str = "mix_out"):
@@ -383,7 +399,7 @@ class RGLRUMixer(Mixer):
         ops.head_linear(u, self.block, self.w_gates, gates, 2 * self.block, ctx.stream, token_req=ctx.token_req)
         unit = cache.side("unit")
         out = ctx.ws.get("rglru_out", T, self.inner_p, x.dtype)[:, :W]
-        ops.label(self.name + ".scan", 30.0 * T * W, (8.0 + 3 * es) * T * W + 8.0 * min(T, ctx.n_requests) * W)
+        ops.label(self.name + ".unit", 30.0 * T * W, (8.0 + 3 * es) * T * W + 8.0 * min(T, ctx.n_requests) * W)
         ops.rglru_scan(gates, self.r_bias, self.i_bias, self.decay, u, y, unit.state, unit.slots, ctx.token_req,
                        ctx.req_first_token, out, self.block, ctx.stream, singles=ctx.n_single > 0, portions=ctx.n_portion > 0)
         return out
