@@ -648,7 +648,7 @@ MLXB_EXPORT int mlxb_retention_chunks_supported(int K, int V) { return K >= 1 &&
 
 // The runs of two rows and more of a step, bfloat16.  qkv, offsets, freq, half, kscale, state: as in retention_scan;
 // powers: float32 [H, 129]; tiles: int32 [n_tiles, 4] = (first token row, rows up to tile_rows, request, first position);
-// scratch: mlxb_retention_chunks_scratch floats; o: float32 [n_tokens, H*V], or, with gate and gated (bfloat16, V <= 128), the
+// scratch: mlxb_retention_chunks_scratch floats; o: float32 [n_tokens, H*V], or, with gate and gated (bfloat16; V up to 128, or 64 with K > 128), the
 // heads' rows divided by their root mean square and multiplied by silu(gate) in gated.
 MLXB_EXPORT int mlxb_retention_chunks(const void* qkv, int ld, int q_off, int k_off, int v_off, const float* freq, int half,
                                       float kscale, const float* powers, float* state, const int* slots, const int* token_req,
@@ -658,7 +658,7 @@ MLXB_EXPORT int mlxb_retention_chunks(const void* qkv, int ld, int q_off, int k_
                                       cudaStream_t stream) {
   if (n_tiles <= 0 || n_requests <= 0) return 0;
   if (H <= 0 || H > 65535 || !mlxb_retention_chunks_supported(K, V) || n_requests > 65535 || half < 0 || 2 * half > K ||
-      (half && !freq) || tile_rows <= 0 || tile_rows > RC_ROWS || (gate && (!gated || V > 128 || ldg < H * V || ldy < H * V)) ||
+      (half && !freq) || tile_rows <= 0 || tile_rows > RC_ROWS || (gate && (!gated || V > (K <= 128 ? 128 : 64) || ldg < H * V || ldy < H * V)) ||
       (!gate && (!o || ldo < H * V)))
     return mlxb_fail(MLXB_BAD_ARG, "retention_chunks: %d heads of %d x %d, %d pairs turned, tiles of %d rows", H, K, V, half, tile_rows);
   const ChunkArgs p = {(const __nv_bfloat16*)qkv, ld, q_off, k_off, v_off, freq, half, kscale, powers, tiles, tile_rows,

@@ -15,7 +15,8 @@
 // A linear recurrence is associative, so a run is cut into pieces of RG_LEN rows: each thread walks one piece of one
 // channel from zero (end state B, product of decays A, the rows' a and b kept in registers), the pieces' (A, B) are
 // chained through shared memory, and each thread walks its piece once more from the state the chain gives it.  A block
-// takes 32 channels (the lanes) and `blockDim.y` pieces at a time, and goes on along the run.
+// takes RG_CHANNELS neighbouring channels and RG_PIECES pieces at a time, and goes on along the run; the rows of the
+// pieces after these are asked for before these are walked.
 #include "common.cuh"
 
 MLXB_DEFINE_LAST_ERROR()
@@ -30,8 +31,9 @@ __device__ __forceinline__ int run_length_2d(const int* __restrict__ token_req, 
   return n;
 }
 
+constexpr int RG_CHANNELS = 16;    // channels of a block
 constexpr int RG_LEN = 8;          // rows of a piece
-constexpr int RG_PIECES = 16;      // pieces a block walks at a time (of a run of several rows)
+constexpr int RG_PIECES = 32;      // pieces a block walks at a time
 
 template <typename T>
 __device__ __forceinline__ float gelu_y(float v);
@@ -43,19 +45,19 @@ __device__ __forceinline__ float gelu_y<__nv_bfloat16>(float v) { return gelu_ne
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 
 // Columns of the gates' products: channel c of block b = c / n, j = c % n: pr at b * 2n + j, pi at b * 2n + n + j.
+// Requests that bring a single row are left to rglru_row_kernel.
 template <typename T>
-__global__ void __launch_bounds__(32 * RG_PIECES)
+__global__ void __launch_bounds__(RG_CHANNELS * RG_PIECES)
 rglru_scan_kernel(const float* gates, int ldg, const float* __restrict__ br, const float* __restrict__ bi,
                   const float* __restrict__ cdecay, const T* u, int ldu, const T* y, int ldy, float* state,
                   const int* __restrict__ slots, const int* __restrict__ token_req,
-                  const int* __restrict__ req_first_token, T* __restrict__ out, int ldo, int W, int n_block, int min_run,
-                  int max_run) {
-  __shared__ float sA[RG_PIECES][32], sB[RG_PIECES][32];
-  const int lane = threadIdx.x, piece = threadIdx.y, pieces = blockDim.y;
-  const int c = blockIdx.x * 32 + lane, r = blockIdx.y;
+                  const int* __restrict__ req_first_token, T* __restrict__ out, int ldo, int W, int n_block) {
+  __shared__ float2 chain[2][RG_PIECES][RG_CHANNELS];      // (A, B) of a piece; two sets, so that one barrier a round is enough
+  const int lane = threadIdx.x, piece = threadIdx.y;
+  const int c = blockIdx.x * RG_CHANNELS + lane, r = blockIdx.y;
   const int t0 = req_first_token[r], t1 = req_first_token[r + 1];
   const int n = run_length_2d(token_req, t0, t1, r);
-  if (n < min_run || n > max_run) return;
+  if (n < 2) return;
   const bool valid = c < W;
   const int cc = valid ? c : 0;
   const int blk = cc / n_block, j = cc - blk * n_block;
@@ -64,53 +66,54 @@ rglru_scan_kernel(const float* gates, int ldg, const float* __restrict__ br, con
   float carry = *sp;             // written in an earlier step: read before the wait
   pdl_wait();
   pdl_trigger();
-  gates = after_wait(gates);
-  u = after_wait(u);
-  y = after_wait(y);
-  const float* gp = gates + (size_t)blk * 2 * n_block + j;
-  for (int base = 0; base < n; base += pieces * RG_LEN) {
-    const int lo = base + piece * RG_LEN;
-    float a[RG_LEN], b[RG_LEN], yy[RG_LEN];
-    float pr[RG_LEN], pi[RG_LEN], uu[RG_LEN];
+  gates = after_wait(gates) + (size_t)blk * 2 * n_block + j;
+  u = after_wait(u) + cc;
+  y = after_wait(y) + cc;
+  float pr[RG_LEN], pi[RG_LEN];
+  T uu[RG_LEN], yy[RG_LEN];
+  auto fetch = [&](int lo) {
 #pragma unroll
     for (int e = 0; e < RG_LEN; ++e) {
-      const bool in = lo + e < n && valid;
-      const size_t t = (size_t)(t0 + (in ? lo + e : 0));
-      pr[e] = in ? gp[t * ldg] : 0.f;
-      pi[e] = in ? gp[t * ldg + n_block] : 0.f;
-      uu[e] = in ? to_f(u[t * ldu + cc]) : 0.f;
-      yy[e] = in ? to_f(y[t * ldy + cc]) : 0.f;
+      const size_t t = (size_t)(t0 + min(lo + e, n - 1));
+      pr[e] = gates[t * ldg];
+      pi[e] = gates[t * ldg + n_block];
+      uu[e] = u[t * ldu];
+      yy[e] = y[t * ldy];
     }
+  };
+  int set = 0;
+  fetch(piece * RG_LEN);
+  for (int base = 0; base < n; base += RG_PIECES * RG_LEN, set ^= 1) {
+    const int lo = base + piece * RG_LEN;
+    float a[RG_LEN], b[RG_LEN], g[RG_LEN];
     float A = 1.f, B = 0.f;
 #pragma unroll
     for (int e = 0; e < RG_LEN; ++e) {
+      const float x = expm1f(sigmoid_f(pr[e] + b_r) * cd);
       const bool in = lo + e < n;
-      const float la = sigmoid_f(pr[e] + b_r) * cd;
-      const float x = expm1f(la);
       a[e] = in ? 1.f + x : 1.f;
-      b[e] = in ? sqrtf(-x * (2.f + x)) * (sigmoid_f(pi[e] + b_i) * uu[e]) : 0.f;
+      b[e] = in ? sqrtf(-x * (2.f + x)) * (sigmoid_f(pi[e] + b_i) * to_f(uu[e])) : 0.f;
+      g[e] = gelu_y<T>(to_f(yy[e]));
       A *= a[e];
       B = fmaf(a[e], B, b[e]);
     }
-    float S = carry;
-    if (pieces > 1) {
-      __syncthreads();
-      sA[piece][lane] = A;
-      sB[piece][lane] = B;
-      __syncthreads();
-      float s = carry;
-      for (int p = 0; p < pieces; ++p) {
-        if (p == piece) S = s;
-        s = fmaf(sA[p][lane], s, sB[p][lane]);
-      }
-      carry = s;
+    chain[set][piece][lane] = make_float2(A, B);
+    const int next = lo + RG_PIECES * RG_LEN;
+    if (base + RG_PIECES * RG_LEN < n) fetch(next);
+    __syncthreads();
+    float S = carry, s = carry;
+#pragma unroll 8
+    for (int p = 0; p < RG_PIECES; ++p) {
+      if (p == piece) S = s;
+      const float2 ab = chain[set][p][lane];
+      s = fmaf(ab.x, s, ab.y);
     }
+    carry = s;
 #pragma unroll
     for (int e = 0; e < RG_LEN; ++e) {
       S = fmaf(a[e], S, b[e]);
-      if (lo + e < n && valid) out[(size_t)(t0 + lo + e) * ldo + c] = from_f<T>(S * gelu_y<T>(yy[e]));
+      if (lo + e < n && valid) out[(size_t)(t0 + lo + e) * ldo + c] = from_f<T>(S * g[e]);
     }
-    if (pieces == 1) carry = S;
   }
   if (piece == 0 && valid) *sp = carry;
 }
@@ -156,9 +159,9 @@ MLXB_EXPORT int mlxb_rglru_scan(int dtype, const float* gates, int ldg, const fl
   if (dtype != MLXB_F32 && dtype != MLXB_BF16) return mlxb_fail(MLXB_BAD_DTYPE, "rglru_scan: dtype code %d", dtype);
 #define RG_GO(T)                                                                                                      \
   if (portions)                                                                                                       \
-    launch_pdl(rglru_scan_kernel<T>, dim3((W + 31) / 32, n_requests), dim3(32, RG_PIECES), 0, stream, gates, ldg, br, bi, \
-               cdecay, (const T*)u, ldu, (const T*)y, ldy, state, slots, token_req, req_first_token, (T*)out, ldo, W, n_block, \
-               2, 0x7fffffff);                                                                                        \
+    launch_pdl(rglru_scan_kernel<T>, dim3((W + RG_CHANNELS - 1) / RG_CHANNELS, n_requests), dim3(RG_CHANNELS, RG_PIECES), 0, \
+               stream, gates, ldg, br, bi, cdecay, (const T*)u, ldu, (const T*)y, ldy, state, slots, token_req,       \
+               req_first_token, (T*)out, ldo, W, n_block);                                                     \
   if (singles)                                                                                                        \
     launch_pdl(rglru_row_kernel<T>, dim3((W + 127) / 128, n_requests), dim3(128), 0, stream, gates, ldg, br, bi, cdecay, \
                (const T*)u, ldu, (const T*)y, ldy, state, slots, token_req, req_first_token, (T*)out, ldo, W, n_block)

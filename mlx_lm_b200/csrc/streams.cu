@@ -65,7 +65,7 @@ __device__ __forceinline__ void norm_row(const float* u, float ss, const float* 
 }
 
 template <typename TO, int SM, int VEC>
-__global__ void streams_read_kernel(const float* x, int ldx, const int* __restrict__ rows, int n_src_rows, int S,
+__global__ void __launch_bounds__(512) streams_read_kernel(const float* x, int ldx, const int* __restrict__ rows, int n_src_rows, int S,
                                     const float* __restrict__ in, const float* __restrict__ w, float eps,
                                     TO* __restrict__ h, int ldh, int D) {
   extern __shared__ __align__(16) float u[];
@@ -105,7 +105,7 @@ __global__ void streams_read_kernel(const float* x, int ldx, const int* __restri
 }
 
 template <typename TO, int SM, int VEC>
-__global__ void streams_update_kernel(float* x, int ldx, const float* y, int ldy, int S, const float* __restrict__ mix,
+__global__ void __launch_bounds__(512) streams_update_kernel(float* x, int ldx, const float* y, int ldy, int S, const float* __restrict__ mix,
                                       const float* __restrict__ out, const int* __restrict__ token_req,
                                       const float* __restrict__ in, const float* __restrict__ w, float eps,
                                       TO* __restrict__ h, int ldh, int D) {

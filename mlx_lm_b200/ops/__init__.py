@@ -1037,6 +1037,11 @@ def retention_chunks_supported(dtype, dim: int, tile_rows: int = 0) -> bool:
     return dtype == torch.bfloat16 and 1 <= dim <= 256 and (tile_rows or PREFILL_TILE) <= RETENTION_TILE
 
 
+def retention_chunks_gated(dim: int, vdim: int) -> bool:
+    """Whether ``retention_chunks`` can norm and gate a head's rows itself (one thread block has all columns of the head)."""
+    return vdim <= (128 if dim <= 128 else 64)
+
+
 def retention_chunks_scratch(n_tokens: int, n_requests: int, n_heads: int, dim: int, vdim: int, tile_rows: int = 0) -> int:
     """Floats of scratch memory ``retention_chunks`` needs: a state per tile of a run."""
     return (n_tokens // (tile_rows or PREFILL_TILE) + n_requests + 1) * n_heads * dim * vdim
@@ -1049,7 +1054,7 @@ def retention_chunks(qkv, q_off: int, k_off: int, v_off: int, freq, kscale: floa
     a tile's contribution to the state, the states along each run, the tiles' outputs.  ``powers``: float32
     ``[heads, RETENTION_TILE + 1]``, the powers 0, 1, .. of every head's decay; ``tiles``: int32 ``[n_tiles, 4]`` = (first token
     row, rows, request, first position), at most ``tile_rows`` rows each.  ``out``: float32 ``[T, heads*V]``; or, with ``gate``
-    and ``gated`` (bfloat16 ``[T, heads*V]``, at most 128 value columns a head), every head's row divided by its root mean
+    and ``gated`` (bfloat16 ``[T, heads*V]``, heads that ``retention_chunks_gated`` takes), every head's row divided by its root mean
     square (``eps`` inside the root) and multiplied by ``silu(gate)``."""
     _need(qkv, torch.bfloat16, "retention_chunks qkv")
     _need(state, torch.float32, "retention_chunks state")

@@ -306,7 +306,7 @@ class RetentionMixer(Mixer):
         where = (ctx.token_req, ctx.req_first_token)
         tiled = (ctx.n_portion > 0 and ctx.portion_tiles is not None and ops.retention_chunks_supported(x.dtype, self.dim))
         cost = (6.0 * T * VW * self.dim, x.element_size() * T * (v_off + VW) + 8.0 * min(T, ctx.n_requests) * VW * self.dim)
-        fused = tiled and ctx.n_single == 0 and self.vdim <= 128      # the tiles' own kernel norms and gates their rows
+        fused = tiled and ctx.n_single == 0 and ops.retention_chunks_gated(self.dim, self.vdim)      # the tiles' own kernel norms and gates their rows
         o = None if fused else ctx.ws.get("retention_o", T, VW, torch.float32)
         if tiled:
             scratch = ctx.ws.flat("retention_states", ops.retention_chunks_scratch(T, ctx.n_requests, H, self.dim, self.vdim),

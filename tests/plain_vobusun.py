@@ -162,7 +162,9 @@ def layers(config, w, tokens, dtype=torch.float64):
     tokens = torch.as_tensor(tokens, dtype=torch.long)
     eps, m = config["norm"]["eps"], config["residual_mult"]
     e = embedding(tokens, w, config, dtype)
-    x = torch.stack([e] * config["streams"])
+    several = config.get("streams") is not None
+    x = torch.stack([e] * (config["streams"] if several else 1))
+    one = torch.ones(1)
     after = []
     for i, layer in enumerate(config["layers"]):
         p = f"l{layer.get('weights_of', i)}"
@@ -171,9 +173,9 @@ def layers(config, w, tokens, dtype=torch.float64):
             sub.append(lambda z: bounded_unit(z, w, p + ".mlp", layer["mlp"]["limit"]))
         for n, f in enumerate(sub, start=1):
             hc = f"{p}.hc{n}"
-            u = read_streams(x, w[hc + ".in"])
+            u = read_streams(x, w[hc + ".in"] if several else one)
             y = f(rms(u, eps) * w[f"{p}.norm{n}"].to(dtype))
-            x = mix_streams(x, w[hc + ".mix"], w[hc + ".out"], y, m)
+            x = mix_streams(x, w[hc + ".mix"], w[hc + ".out"], y, m) if several else x + m * y
         after.append(x.sum(dim=0))
     x = x.sum(dim=0)
     logits = (rms(x, eps) * w["final.norm"].to(dtype)) @ w["head"].to(dtype).T
