@@ -104,53 +104,53 @@ __global__ void embed_pairs_kernel(const int* __restrict__ tok, const int* __res
                                    long long mul_prev, long long mul_cur, float eps, int* __restrict__ status) {
   extern __shared__ float row[];      // the sum before the norm
   __shared__ float red[33];
-  __shared__ int s_prev;
+  const int t = blockIdx.x;
+  const int r = token_req[t], p = pos[t];
+  int t0 = 0, t1 = 0, slot = 0;
+  if (r >= 0) { t0 = req_first_token[r]; t1 = req_first_token[r + 1]; slot = slots[r]; }
+  const bool first = r >= 0 && t == t0;
   pdl_wait();
   pdl_trigger();
-  const int t = blockIdx.x;
   float* o = out + (size_t)t * S * D;
-  const int r = token_req[t];
   const int id = tok[t];
+  long long prev = 0;
+  if (pairs && r >= 0 && p > 0) prev = first ? (long long)after_wait(last)[slot] : (long long)tok[t - 1];
   bool ok = r >= 0;
   if (ok && (id < 0 || id >= V)) { ok = false; if (threadIdx.x == 0) atomicOr(status, MLXB_ST_TOKEN_RANGE); }
-  const bool first = r >= 0 && t == req_first_token[r];
+  if (!ok) {
+    for (int d = threadIdx.x; d < S * D; d += blockDim.x) o[d] = 0.f;
+  } else {
+    const T* e = wte + (size_t)id * D;
+    const T* b = nullptr;
+    if (pairs) {
+      long long at = buckets;
+      if (p > 0) {
+        at = (prev * mul_prev + (long long)id * mul_cur) % buckets;
+        if (at < 0) at += buckets;
+      }
+      b = pairs + (size_t)at * D;
+    }
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+      float v = to_f(e[d]) * scale;
+      if (b) v += to_f(b[d]);
+      row[d] = v;
+      ss = fmaf(v, v, ss);
+    }
+    const float rinv = w ? 1.f / sqrtf(block_sum(ss, red) / (float)D + eps) : 1.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+      const float v = w ? row[d] * rinv * w[d] : row[d];
+      for (int n = 0; n < S; ++n) o[(size_t)n * D + d] = v;
+    }
+  }
   if (pairs && first) {
-    if (threadIdx.x == 0) s_prev = pos[t] > 0 ? (int)after_wait(last)[slots[r]] : -1;
-    // the run's last row: its rows come first in the request's range
-    const int t1 = req_first_token[r + 1];
+    // the run's last row (a request's rows come first in its range); every thread has read the slot by the first barrier
     int n = 0;
     for (int base = t; base < t1; base += blockDim.x) {
       const int tt = base + threadIdx.x;
       n += __syncthreads_count(tt < t1 && token_req[tt] == r);
     }
-    if (threadIdx.x == 0) last[slots[r]] = (float)tok[t + n - 1];
-  }
-  if (!ok) {
-    for (int d = threadIdx.x; d < S * D; d += blockDim.x) o[d] = 0.f;
-    return;
-  }
-  const T* e = wte + (size_t)id * D;
-  const T* b = nullptr;
-  if (pairs) {
-    const int prev = first ? s_prev : tok[t - 1];      // (s_prev: written before the barriers above)
-    long long at = buckets;
-    if (!first || pos[t] > 0) {
-      at = ((long long)prev * mul_prev + (long long)id * mul_cur) % buckets;
-      if (at < 0) at += buckets;
-    }
-    b = pairs + (size_t)at * D;
-  }
-  float ss = 0.f;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
-    float v = to_f(e[d]) * scale;
-    if (b) v += to_f(b[d]);
-    row[d] = v;
-    ss = fmaf(v, v, ss);
-  }
-  const float rinv = w ? 1.f / sqrtf(block_sum(ss, red) / (float)D + eps) : 1.f;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
-    const float v = w ? row[d] * rinv * w[d] : row[d];
-    for (int n = 0; n < S; ++n) o[(size_t)n * D + d] = v;
+    if (threadIdx.x == 0) last[slot] = (float)tok[t + n - 1];
   }
 }
 

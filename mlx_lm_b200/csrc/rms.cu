@@ -7,8 +7,8 @@
 //                  from one (offset 1).  A gate g (activation dtype) may come in: mode 1 multiplies x by
 //                  silu(g) BEFORE the statistics, mode 2 multiplies the normed value by silu(g).
 //                  x is float32 or has the activation dtype, which the result has.  No weight: the normed value as it is
-//                  (times the offset where there is one).  All arithmetic is float32.  Rows or parts of up to 512
-//                  columns (heads) take a kernel with a warp each.
+//                  (times the offset where there is one).  All arithmetic is float32.  Rows or parts of up to
+//                  512 columns without a weight, or in the activation dtype, take a kernel with a warp each.
 // residual_update  x[r, :] += scale * (f1(y1[r, :]) + f2(y2[r, :])),  f_i = rmsnorm with weight w_i over the
 //                  whole row, or the identity where w_i is null; y2 may be null.  Optionally a copy of the new
 //                  row in the activation dtype is left in `cast_out` for the products that read it next.
@@ -137,7 +137,8 @@ MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, int x_f32, const void* x, int ldx, c
   if (out_dtype != MLXB_F32 && out_dtype != MLXB_BF16) return mlxb_fail(MLXB_BAD_DTYPE, "rmsnorm: dtype code %d", out_dtype);
   const int Dg = D / groups;
   const int xb = (x_f32 || out_dtype == MLXB_F32) ? 16 : 8, ob = out_dtype == MLXB_F32 ? 16 : 8;   // bytes of four columns
-  const bool parts = rows == nullptr && Dg % 4 == 0 && Dg <= 128 * RP_STEPS && ldx % 4 == 0 && ldo % 4 == 0 &&
+  // (weighted norms of float32 rows keep the block per row or part and its order of additions)
+  const bool parts = (w == nullptr || (!x_f32 && out_dtype == MLXB_BF16)) && rows == nullptr && Dg % 4 == 0 && Dg <= 128 * RP_STEPS && ldx % 4 == 0 && ldo % 4 == 0 &&
                      (!gate || ldg % 4 == 0) && (uintptr_t)x % xb == 0 && ((uintptr_t)out | (uintptr_t)gate) % ob == 0;
   const int threads = parts ? 256 : (Dg >= 2048 ? 256 : (Dg >= 512 ? 128 : (Dg >= 128 ? 64 : 32)));
   const dim3 grid = parts ? dim3((unsigned)(((long long)R * groups + 7) / 8)) : dim3(R, groups);
