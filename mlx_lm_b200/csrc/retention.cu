@@ -230,23 +230,36 @@ __device__ __forceinline__ void stage_turned(const __nv_bfloat16* src, int ld, i
   const int tid = threadIdx.x, nt = blockDim.x;
   if (VEC) {
     const int per = (K - half) / 4;      // four neighbouring pairs, or four dimensions that do not turn
-    for (int e = tid; e < rows * per; e += nt) {
-      const int tok = e / per, i = (e - tok * per) * 4;
-      __nv_bfloat16* ph = hi + tok * lds;
-      __nv_bfloat16* pl = lo + tok * lds;
-      float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
-      const bool turn = i < half;
-      if (tok < n) {
-        const __nv_bfloat16* rp = src + (size_t)(row0 + tok) * ld;
-        const float f = fall ? scale * fall[fall_last - tok] : scale;
-        const uint2 ub = *reinterpret_cast<const uint2*>(rp + i + half);
-        const float v1[4] = {__uint_as_float(ub.x << 16), __uint_as_float(ub.x & 0xffff0000u), __uint_as_float(ub.y << 16),
-                             __uint_as_float(ub.y & 0xffff0000u)};
-        if (turn) {
-          const uint2 ua = *reinterpret_cast<const uint2*>(rp + i);
-          const float v0[4] = {__uint_as_float(ua.x << 16), __uint_as_float(ua.x & 0xffff0000u), __uint_as_float(ua.y << 16),
-                               __uint_as_float(ua.y & 0xffff0000u)};
+    constexpr int UN = 4;                // items whose loads are in flight together
+    for (int e0 = tid; e0 < rows * per; e0 += UN * nt) {
+      uint2 ua[UN], ub[UN];
+#pragma unroll
+      for (int x = 0; x < UN; ++x) {
+        const int e = e0 + x * nt, tok = e / per, i = (e - tok * per) * 4;
+        ua[x] = ub[x] = make_uint2(0u, 0u);
+        if (tok < n) {                   // (an item beyond the last has a row beyond n)
+          const __nv_bfloat16* rp = src + (size_t)(row0 + tok) * ld;
+          ub[x] = *reinterpret_cast<const uint2*>(rp + i + half);
+          if (i < half) ua[x] = *reinterpret_cast<const uint2*>(rp + i);
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < UN; ++x) {
+        const int e = e0 + x * nt;
+        if (e >= rows * per) break;
+        const int tok = e / per, i = (e - tok * per) * 4;
+        __nv_bfloat16* ph = hi + tok * lds;
+        __nv_bfloat16* pl = lo + tok * lds;
+        const float f = fall ? (tok < n ? scale * fall[fall_last - tok] : 0.f) : scale;
+        const float v1[4] = {__uint_as_float(ub[x].x << 16), __uint_as_float(ub[x].x & 0xffff0000u),
+                             __uint_as_float(ub[x].y << 16), __uint_as_float(ub[x].y & 0xffff0000u)};
+        float b[4];
+        uint2 h, l;
+        if (i < half) {
+          const float v0[4] = {__uint_as_float(ua[x].x << 16), __uint_as_float(ua[x].x & 0xffff0000u),
+                               __uint_as_float(ua[x].y << 16), __uint_as_float(ua[x].y & 0xffff0000u)};
           const float fp = (float)(pos0 + tok);
+          float a[4];
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             float sn, cs;
@@ -254,21 +267,18 @@ __device__ __forceinline__ void stage_turned(const __nv_bfloat16* src, int ld, i
             a[q] = (v0[q] * cs - v1[q] * sn) * f;
             b[q] = (v1[q] * cs + v0[q] * sn) * f;
           }
+          mb_split2(a[0], a[1], h.x, l.x);
+          mb_split2(a[2], a[3], h.y, l.y);
+          *reinterpret_cast<uint2*>(ph + i) = h;
+          *reinterpret_cast<uint2*>(pl + i) = l;
         } else {
 #pragma unroll
           for (int q = 0; q < 4; ++q) b[q] = v1[q] * f;
         }
-      }
-      uint2 h, l;
-      mb_split2(b[0], b[1], h.x, l.x);
-      mb_split2(b[2], b[3], h.y, l.y);
-      *reinterpret_cast<uint2*>(ph + i + half) = h;
-      *reinterpret_cast<uint2*>(pl + i + half) = l;
-      if (turn) {
-        mb_split2(a[0], a[1], h.x, l.x);
-        mb_split2(a[2], a[3], h.y, l.y);
-        *reinterpret_cast<uint2*>(ph + i) = h;
-        *reinterpret_cast<uint2*>(pl + i) = l;
+        mb_split2(b[0], b[1], h.x, l.x);
+        mb_split2(b[2], b[3], h.y, l.y);
+        *reinterpret_cast<uint2*>(ph + i + half) = h;
+        *reinterpret_cast<uint2*>(pl + i + half) = l;
       }
     }
   } else {
@@ -306,6 +316,7 @@ __device__ __forceinline__ void stage_values(const __nv_bfloat16* src, int ld, i
                                              __nv_bfloat16* sv, int lds) {
   if (VEC) {
     const int per = VS / 8;
+#pragma unroll 4
     for (int e = threadIdx.x; e < rows * per; e += blockDim.x) {
       const int tok = e / per, c = (e - tok * per) * 8;
       uint4 u = make_uint4(0u, 0u, 0u, 0u);
@@ -342,7 +353,7 @@ __device__ __forceinline__ size_t chunk_slot(const ChunkArgs& p, int r, int pos)
 // A tile's contribution to the state, columns v0 .. v0 + 63 of one head: warp w takes v rows 16 (w % 4) .. and half of
 // the K columns.
 template <int KP, bool VEC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, KP <= 64 ? 3 : 1)
 retention_chunk_states_kernel(const ChunkArgs p) {
   extern __shared__ __align__(16) unsigned char rc_raw[];
   constexpr int LK = KP + 8, LV = 64 + 8;
@@ -482,6 +493,7 @@ retention_chunk_out_kernel(const ChunkArgs p, float* __restrict__ o, int ldo, co
   stage_turned<VEC>(qkv + p.q_off + (size_t)h * p.K, p.ld, t0, n, rows, pos, p.freq, p.half, p.K, KP, 1.f, nullptr, 0, qh, ql, LK);
   // S^T: rows v, columns k
   if (VEC) {
+#pragma unroll 8
     for (int e = threadIdx.x; e < VS * (KP / 4); e += blockDim.x) {
       const int v = e / (KP / 4), c = (e - v * (KP / 4)) * 4;
       float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
