@@ -2,8 +2,8 @@
 // token): what stands around the attention kernel.
 //
 // latent_prepare  From a token's queries and its down projection (columns of one fused projection, or rows of two
-//                 buffers where the queries come out of a product of their own): `down` holds R latent columns and dr columns of a
-//                 rotated key part that all heads share.  The latent columns are divided by their root mean square
+//                 buffers where the queries come out of a product of their own): `down` holds R latent columns and dr
+//                 columns of a rotated key part that all heads share.  The latent columns are divided by their root mean square
 //                 and multiplied by a weight (c); the key part is rotated by the position; [c | rotated part | 0..]
 //                 becomes the token's row in the pages (one "head", Dh >= R + dr wide).  Of every query head
 //                 ([d unrotated | dr rotated] in the projection) the rotated part is rotated the same way and put,
@@ -20,7 +20,8 @@
 MLXB_DEFINE_LAST_ERROR()
 
 template <typename T>
-__global__ void latent_prepare_kernel(const T* queries, int ldqs, const T* proj, int ld, int q_off, int c_off, int H, int d, int dr, int R,
+__global__ void latent_prepare_kernel(const T* queries, int ldqs, const T* proj, int ld, int q_off, int c_off, int H,
+                                      int d, int dr, int R,
                                       const float* __restrict__ w, float eps, const float* __restrict__ freq,
                                       int interleaved, const int* __restrict__ positions,
                                       const int* __restrict__ token_req, const int* __restrict__ block_table,
@@ -83,7 +84,8 @@ __global__ void latent_prepare_kernel(const T* queries, int ldqs, const T* proj,
 }
 
 // queries: head h's columns from q_off + h * (d + dr) of rows at stride ldqs; proj: the down projection from c_off.
-MLXB_EXPORT int mlxb_latent_prepare(int dtype, const void* queries, int ldqs, const void* proj, int ld, int q_off, int c_off, int H, int d, int dr, int R,
+MLXB_EXPORT int mlxb_latent_prepare(int dtype, const void* queries, int ldqs, const void* proj, int ld, int q_off,
+                                    int c_off, int H, int d, int dr, int R,
                                     const float* w, float eps, const float* freq, int interleaved, const int* positions,
                                     const int* token_req, const int* block_table, int max_pages, int n_pages, int page,
                                     int Dh, void* pool, int write, float* q_lat, int ldq, int qhs, int n_tokens,
@@ -98,7 +100,8 @@ MLXB_EXPORT int mlxb_latent_prepare(int dtype, const void* queries, int ldqs, co
                Dh, (float*)pool, write, q_lat, ldq, qhs, status, mscale);
   else if (dtype == MLXB_BF16)
     launch_pdl(latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream,
-               (const __nv_bfloat16*)queries, ldqs, (const __nv_bfloat16*)proj, ld, q_off, c_off, H, d, dr, R, w, eps, freq, interleaved, positions, token_req,
+               (const __nv_bfloat16*)queries, ldqs, (const __nv_bfloat16*)proj, ld, q_off, c_off, H, d, dr, R, w, eps, freq,
+               interleaved, positions, token_req,
                block_table, max_pages, n_pages, page, Dh, (__nv_bfloat16*)pool, write, q_lat, ldq, qhs, status, mscale);
   else
     return mlxb_fail(MLXB_BAD_DTYPE, "latent_prepare: dtype code %d", dtype);
