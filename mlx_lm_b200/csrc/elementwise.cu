@@ -6,6 +6,7 @@
 //   xielu           out[t, j] = f(in[t, j]) with two learned numbers (a, b) of the layer, read from device memory:
 //                   z > 0: softplus(a) z^2 + z/2;  z <= 0: (1/2 + softplus(b)) (exp(z) - 1 - z) + z/2.  In place if out = in.
 //   join_rows       out[t] = [a[t] | b[t]] in the activation dtype from float32 rows (b may be null: a plain cast).
+//   soft_cap        x <- cap * tanh(x / cap) in place on float32 rows.
 #include "common.cuh"
 #include "gated_unit.cuh"
 
@@ -204,4 +205,31 @@ MLXB_EXPORT int mlxb_xielu(int dtype, const void* in, int ldi, void* out, int ld
   else
     return mlxb_fail(MLXB_BAD_DTYPE, "xielu: dtype code %d", dtype);
   return mlxb_check_launch("xielu");
+}
+
+// x: float32, n elements one after the other, 16-byte aligned.
+__global__ void soft_cap_kernel(float* x, long long n, float cap) {
+  pdl_wait();
+  pdl_trigger();
+  x = after_wait(x);
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i + 4 <= n) {
+    float4 v = *reinterpret_cast<const float4*>(x + i);
+    v.x = cap * tanhf(v.x / cap);
+    v.y = cap * tanhf(v.y / cap);
+    v.z = cap * tanhf(v.z / cap);
+    v.w = cap * tanhf(v.w / cap);
+    *reinterpret_cast<float4*>(x + i) = v;
+  } else {
+    for (long long j = i; j < n; ++j) x[j] = cap * tanhf(x[j] / cap);
+  }
+}
+
+MLXB_EXPORT int mlxb_soft_cap(float* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f) || ((uintptr_t)x & 15)) return mlxb_fail(MLXB_BAD_ARG, "soft_cap: %lld elements, cap %g", n, (double)cap);
+  const int threads = 256;
+  const dim3 grid((unsigned)((n + 4 * threads - 1) / (4 * threads)));
+  launch_pdl(soft_cap_kernel, grid, dim3(threads), 0, stream, x, n, cap);
+  return mlxb_check_launch("soft_cap");
 }

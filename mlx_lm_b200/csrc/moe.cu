@@ -6,13 +6,13 @@
 //             correction per expert added to the scores for the choice only; groups of neighbouring experts of which
 //             only the best few stay in the race; identity experts (no tensors; marked -2); weights scaled.
 // moe_combine x[t] += the sum of the token's choices' rows, an identity expert's choice being its weight times the input.
-// moe_plan    one CTA: the (token, choice) slots sorted by expert, and a list of tiles of at most `tile_rows` slots of
+// moe_plan    (moe_plan_table: for experts that a table of the token ids names, without a router) one CTA: the (token, choice) slots sorted by expert, and a list of tiles of at most `tile_rows` slots of
 //             one expert each: tile_info[i] = (expert, first place in the sorted list, slots).  How many tiles there are
 //             depends on the data; the kernels that follow are launched for the most there can be and read the count.
 // moe_gemm    per tile and block of output columns: out[slot, n] = sum_k A[row(slot), k] W[expert][n, k], the rows
 //             gathered through the sorted list (row(slot) = slot / a_div: the token's row where the input is shared by
 //             a token's choices, the slot's own row where it is not).  GATED: W holds [gate | up] rows (2 N of them);
-//             with the routing weight w of the slot the result is silu(w g) * (w u), which is what the gated unit
+//             with the routing weight w of the slot (1 where no weights are given) the result is silu(w g) * (w u), which is what the gated unit
 //             makes of the expert's input scaled by w (the products are linear in it, so w is applied to the float32
 //             sums instead of to the rounded input), or the bounded unit times w (gated_unit.cuh).  bfloat16 runs on tensor cores (mma.sync m16n8k16, float32
 //             accumulation; 64 x 64 tiles, 16-byte cp.async in two stages), float32 (and inner sizes that are no
@@ -192,23 +192,51 @@ MLXB_EXPORT int mlxb_moe_combine(int dtype, float* x, int ldx, const float* y, i
   return mlxb_check_launch("moe_combine");
 }
 
-// sorted [S]; tile_info [max_tiles][3]; n_tiles [1].  Shared memory: 3 E + 1 ints.
-__global__ void moe_plan_kernel(const int* sel_expert, int S, int E, int tile_rows, int max_tiles,
+// Where the slots' experts come from: what moe_route chose, or a table with a row of `top` experts per token id.
+struct MoeChosen {
+  const int* sel_expert;
+  __device__ __forceinline__ void arrived() { sel_expert = after_wait(sel_expert); }
+  __device__ __forceinline__ int operator()(int i) const { return sel_expert[i]; }
+};
+struct MoeTable {
+  const int *tokens, *token_req, *table;
+  int top, vocab;
+  int* status;
+  __device__ __forceinline__ void arrived() {}
+  __device__ __forceinline__ int operator()(int i) const {
+    const int t = i / top;
+    if (token_req && token_req[t] < 0) return -1;
+    const int id = tokens[t];
+    if (id < 0 || id >= vocab) { atomicOr(status, MLXB_ST_TOKEN_RANGE); return -1; }
+    return table[(size_t)id * top + (i - t * top)];
+  }
+};
+
+// sorted [S]; tile_info [max_tiles][3]; n_tiles [1].  Shared memory: 3 E + 1 ints.  EARLY: the experts follow from the step's
+// inputs and are counted before the wait for the kernel before.
+template <typename Source, bool EARLY>
+__global__ void moe_plan_kernel(Source expert_of, int S, int E, int tile_rows, int max_tiles,
                                 int* __restrict__ sorted, int* __restrict__ tile_info, int* __restrict__ n_tiles) {
   extern __shared__ int mp_smem[];
   int* cnt = mp_smem;          // [E]
   int* off = cnt + E;          // [E]
   int* cur = off + E;          // [E]
   for (int e = threadIdx.x; e < E; e += blockDim.x) { cnt[e] = 0; cur[e] = 0; }
-  pdl_wait();
-  pdl_trigger();
-  sel_expert = after_wait(sel_expert);
+  if (!EARLY) {
+    pdl_wait();
+    pdl_trigger();
+    expert_of.arrived();
+  }
   __syncthreads();
   for (int i = threadIdx.x; i < S; i += blockDim.x) {
-    const int e = sel_expert[i];
+    const int e = expert_of(i);
     if (e >= 0 && e < E) atomicAdd(&cnt[e], 1);
   }
   __syncthreads();
+  if (EARLY) {
+    pdl_wait();                // the tiles below may still be read by the products before
+    pdl_trigger();
+  }
   if (threadIdx.x == 0) {
     int acc = 0, nt = 0;
     for (int e = 0; e < E; ++e) {
@@ -225,19 +253,38 @@ __global__ void moe_plan_kernel(const int* sel_expert, int S, int E, int tile_ro
   }
   __syncthreads();
   for (int i = threadIdx.x; i < S; i += blockDim.x) {
-    const int e = sel_expert[i];
+    const int e = expert_of(i);
     if (e >= 0 && e < E) sorted[off[e] + atomicAdd(&cur[e], 1)] = i;
   }
+}
+
+static int moe_plan_check(int S, int E, int tile_rows, int max_tiles) {
+  if (E <= 0 || tile_rows <= 0 || max_tiles < (S + tile_rows - 1) / tile_rows + E || E > 4096)
+    return mlxb_fail(MLXB_BAD_ARG, "moe_plan: %d slots, %d experts, tiles of %d, room for %d", S, E, tile_rows, max_tiles);
+  return 0;
 }
 
 MLXB_EXPORT int mlxb_moe_plan(const int* sel_expert, int S, int E, int tile_rows, int max_tiles, int* sorted,
                               int* tile_info, int* n_tiles, cudaStream_t stream) {
   if (S <= 0) return 0;
-  if (E <= 0 || tile_rows <= 0 || max_tiles < (S + tile_rows - 1) / tile_rows + E || E > 8192)
-    return mlxb_fail(MLXB_BAD_ARG, "moe_plan: %d slots, %d experts, tiles of %d, room for %d", S, E, tile_rows, max_tiles);
-  launch_pdl(moe_plan_kernel, dim3(1), dim3(S >= 4096 ? 1024 : 256), sizeof(int) * 3 * (size_t)E, stream, sel_expert, S,
-             E, tile_rows, max_tiles, sorted, tile_info, n_tiles);
+  if (int e = moe_plan_check(S, E, tile_rows, max_tiles)) return e;
+  launch_pdl(moe_plan_kernel<MoeChosen, false>, dim3(1), dim3(S >= 4096 ? 1024 : 256), sizeof(int) * 3 * (size_t)E, stream,
+             MoeChosen{sel_expert}, S, E, tile_rows, max_tiles, sorted, tile_info, n_tiles);
   return mlxb_check_launch("moe_plan");
+}
+
+// The plan of a feed-forward without a router: token t's experts are row tokens[t] of `table` (int32 [vocab, top]); rows whose
+// token_req is negative take no part.  A token id outside the table sets a status bit.
+MLXB_EXPORT int mlxb_moe_plan_table(const int* tokens, const int* token_req, const int* table, int vocab, int top, int T, int E,
+                                    int tile_rows, int max_tiles, int* sorted, int* tile_info, int* n_tiles, int* status,
+                                    cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const int S = T * top;
+  if (top <= 0 || vocab <= 0 || !table) return mlxb_fail(MLXB_BAD_ARG, "moe_plan: a table of %d rows of %d experts", vocab, top);
+  if (int e = moe_plan_check(S, E, tile_rows, max_tiles)) return e;
+  launch_pdl(moe_plan_kernel<MoeTable, true>, dim3(1), dim3(S >= 1024 ? 1024 : 256), sizeof(int) * 3 * (size_t)E, stream,
+             MoeTable{tokens, token_req, table, top, vocab, status}, S, E, tile_rows, max_tiles, sorted, tile_info, n_tiles);
+  return mlxb_check_launch("moe_plan (table)");
 }
 
 // ---------------------------------------------------------------- CUDA cores: any sizes, float32 or bfloat16 inputs
@@ -295,7 +342,7 @@ moe_gemm_simt_kernel(const T* A, int lda, int a_div, const T* __restrict__ W, lo
   }
   const int slot = sSlot[r];
   if (slot < 0) return;
-  const float w = GATED ? sel_weight[slot] : 1.f;
+  const float w = GATED && sel_weight ? sel_weight[slot] : 1.f;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int n = n0 + cb + 16 * i;
@@ -380,7 +427,7 @@ moe_rows_kernel(const __nv_bfloat16* A, int lda, int a_div, const __nv_bfloat16*
         for (int rr = 0; rr < MV_ROWS; ++rr)
           if (rr == lane) { v = acc[0][rr]; v2 = acc[GATED ? 1 : 0][rr]; }
         if (GATED) {
-          v = mlxb_gated_unit(act, v, v2, sel_weight[slot], limit);
+          v = mlxb_gated_unit(act, v, v2, sel_weight ? sel_weight[slot] : 1.f, limit);
         }
         out[(size_t)slot * ldo + n] = from_f<TO>(v);
       }
@@ -485,7 +532,7 @@ moe_gemm_tc_kernel(const __nv_bfloat16* A, int lda, int a_div, const __nv_bfloat
   for (int half = 0; half < 2; ++half) {
     const int slot = sSlot[warp * 16 + g + half * 8];
     if (slot < 0) continue;
-    const float w = GATED ? sel_weight[slot] : 1.f;
+    const float w = GATED && sel_weight ? sel_weight[slot] : 1.f;
 #pragma unroll
     for (int j = 0; j < MG_BN / 8; ++j)
 #pragma unroll
@@ -511,7 +558,7 @@ MLXB_EXPORT int mlxb_moe_gemm(int dtype, int out_f32, int gated, const void* A, 
                               const int* n_tiles, int max_tiles, int tile_rows, const float* sel_weight, void* out,
                               int ldo, int act, float limit, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
-  if (N <= 0 || K <= 0 || a_div <= 0 || lda < K || ldo < N || (gated && !sel_weight) ||
+  if (N <= 0 || K <= 0 || a_div <= 0 || lda < K || ldo < N ||
       (tile_rows != MG_BM && tile_rows != MS_BM && tile_rows != MV_ROWS) ||
       ((tile_rows == MG_BM || tile_rows == MV_ROWS) && dtype != MLXB_BF16))
     return mlxb_fail(MLXB_BAD_ARG, "moe_gemm: %d x %d, strides %d / %d, tiles of %d rows", N, K, lda, ldo, tile_rows);

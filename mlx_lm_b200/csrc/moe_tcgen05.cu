@@ -193,7 +193,7 @@ moe_gemm_tc05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
       const int r = q * 32 + lane;
       const bool live = r < cnt;
       const int slot = live ? sorted[first + r] : -1;
-      const float wgt = (GATED && live) ? sel_weight[slot] : 1.f;
+      const float wgt = (GATED && live && sel_weight) ? sel_weight[slot] : 1.f;
       if (!mbar_wait(&sm.acc_full[b], (it >> 1) & 1, abort_flag)) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(b * MT_BN);
@@ -380,7 +380,7 @@ MLXB_EXPORT int mlxb_moe_gemm_tc05(int gated, const void* A, int lda, int S, con
                                    cudaStream_t stream) {
   if (max_tiles <= 0 || S <= 0) return 0;
   if (N <= 0 || K <= 0 || E <= 0 || (K & 7) || (N & 7) || (lda & 7) || (ldo & 7) || lda < K || ldo < N ||
-      NW != (gated ? 2 : 1) * N || (gated && !sel_weight) || (((uintptr_t)A | (uintptr_t)W | (uintptr_t)out) & 15) ||
+      NW != (gated ? 2 : 1) * N || (((uintptr_t)A | (uintptr_t)W | (uintptr_t)out) & 15) ||
       (long long)E * NW > 0x7fffffffLL)
     return mlxb_fail(MLXB_BAD_ARG, "moe_gemm (tensor cores): %d experts of %d x %d, strides %d / %d", E, NW, K, lda, ldo);
   MtLaunch l = {{}, {}, sorted, tile_info, n_tiles, NW, N, K, sel_weight, out, ldo, status, max_tiles, stream, act, limit};

@@ -12,6 +12,9 @@
 // residual_update  x[r, :] += scale * (f1(y1[r, :]) + f2(y2[r, :])),  f_i = rmsnorm with weight w_i over the
 //                  whole row, or the identity where w_i is null; y2 may be null.  Optionally a copy of the new
 //                  row in the activation dtype is left in `cast_out` for the products that read it next.
+// norm_update      y = scale * (sum of the row's `terms` rows of y1) + y2[r, :];  x[r, :] += y / sqrt(mean(y^2) + eps) * w: a sublayer
+//                  whose result is normed before it joins the stream, with the sum over the experts a token used in the same
+//                  pass, and a copy of the new row as above.
 #include "common.cuh"
 
 MLXB_DEFINE_LAST_ERROR()
@@ -244,4 +247,121 @@ MLXB_EXPORT int mlxb_head_difference(int out_dtype, const float* a, int lda, con
   else
     return mlxb_fail(MLXB_BAD_DTYPE, "head_difference: dtype code %d", out_dtype);
   return mlxb_check_launch("head_difference");
+}
+
+// VEC: four columns a thread and step (16-byte accesses), or one.  A row's y and x stay in registers: NV * VEC * blockDim.x
+// columns at most.
+template <typename TO, int VEC, int NV>
+__global__ void __launch_bounds__(512)
+norm_update_kernel(float* x, int ldx, const float* y1, int ld1, int terms, float scale, const float* y2, int ld2,
+                   const float* __restrict__ w, float eps, const int* __restrict__ token_req, TO* __restrict__ cast_out, int ldc,
+                   int D) {
+  __shared__ float red[33];
+  const int r = blockIdx.x;
+  if (token_req && token_req[r] < 0) return;
+  auto get = [](const float* p, float (&v)[VEC]) {
+    if (VEC == 4) {
+      const float4 q = *reinterpret_cast<const float4*>(p);
+      v[0] = q.x; v[VEC > 1 ? 1 : 0] = q.y; v[VEC > 2 ? 2 : 0] = q.z; v[VEC > 3 ? 3 : 0] = q.w;
+    } else {
+      v[0] = *p;
+    }
+  };
+  float wv[NV][VEC], xv[NV][VEC], y[NV][VEC];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * VEC;
+    if (c < D) get(w + c, wv[i]);
+  }
+  pdl_wait();
+  pdl_trigger();
+  x = after_wait(x);
+  y1 = after_wait(y1);
+  y2 = after_wait(y2);
+  float* xr = x + (size_t)r * ldx;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * VEC;
+    if (c < D) {
+      get(xr + c, xv[i]);
+      get(y1 + (size_t)r * terms * ld1 + c, y[i]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[i][e] = 0.f;
+    }
+  }
+  for (int k = 1; k < terms; ++k)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * VEC;
+      if (c < D) {
+        float a[VEC];
+        get(y1 + ((size_t)r * terms + k) * ld1 + c, a);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[i][e] += a[e];
+      }
+    }
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * VEC;
+    float b[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) b[e] = 0.f;
+    if (y2 && c < D) get(y2 + (size_t)r * ld2 + c, b);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      y[i][e] = fmaf(scale, y[i][e], b[e]);
+      s = fmaf(y[i][e], y[i][e], s);
+    }
+  }
+  const float rinv = 1.f / sqrtf(block_sum(s, red) / (float)D + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * VEC;
+    if (c >= D) continue;
+    float n[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) n[e] = xv[i][e] + y[i][e] * rinv * wv[i][e];
+    if (VEC == 4) {
+      store4(xr + c, n);
+      if (cast_out) store4(cast_out + (size_t)r * ldc + c, n);
+    } else {
+      xr[c] = n[0];
+      if (cast_out) cast_out[(size_t)r * ldc + c] = from_f<TO>(n[0]);
+    }
+  }
+}
+
+// x: float32 [R, D] at row stride ldx, in place; y1: float32 [R * terms, D]; y2: float32 [R, D] or null; w: float32 [D];
+// token_req: int32 [R] or null (negative: the row is left alone); cast_out: [R, D] of cast_dtype, or null.
+MLXB_EXPORT int mlxb_norm_update(int cast_dtype, float* x, int ldx, const float* y1, int ld1, int terms, float scale,
+                                 const float* y2, int ld2, const float* w, float eps, const int* token_req, void* cast_out,
+                                 int ldc, int R, int D, cudaStream_t stream) {
+  if (R <= 0) return 0;
+  if (cast_dtype != MLXB_F32 && cast_dtype != MLXB_BF16) return mlxb_fail(MLXB_BAD_DTYPE, "norm_update: dtype code %d", cast_dtype);
+  const int cb = cast_dtype == MLXB_F32 ? 16 : 8;
+  const bool vec = D % 4 == 0 && ldx % 4 == 0 && ld1 % 4 == 0 && (!y2 || ld2 % 4 == 0) && (!cast_out || ldc % 4 == 0) &&
+                   (((uintptr_t)x | (uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)w) & 15) == 0 && (uintptr_t)cast_out % cb == 0;
+  const int n = vec ? D / 4 : D;               // steps of one thread over a row, all together
+  if (D <= 0 || terms <= 0 || ldx < D || ld1 < D || (y2 && ld2 < D) || (cast_out && ldc < D) || n > 512 * 8)
+    return mlxb_fail(MLXB_BAD_ARG, "norm_update: width %d, %d terms, strides %d / %d / %d / %d", D, terms, ldx, ld1, ld2, ldc);
+  int threads = 64;
+  while (threads < 512 && n > threads * 2) threads *= 2;
+  const int nv = (n + threads - 1) / threads;
+#define NU_GO(TO, VEC, NV)                                                                                                \
+  launch_pdl(norm_update_kernel<TO, VEC, NV>, dim3(R), dim3(threads), 0, stream, x, ldx, y1, ld1, terms, scale, y2, ld2, w, \
+             eps, token_req, (TO*)cast_out, ldc, D)
+#define NU_BY(TO, VEC)                    \
+  do {                                    \
+    if (nv <= 1) NU_GO(TO, VEC, 1);       \
+    else if (nv <= 2) NU_GO(TO, VEC, 2);  \
+    else if (nv <= 4) NU_GO(TO, VEC, 4);  \
+    else NU_GO(TO, VEC, 8);               \
+  } while (0)
+  if (cast_dtype == MLXB_F32) { if (vec) NU_BY(float, 4); else NU_BY(float, 1); }
+  else { if (vec) NU_BY(__nv_bfloat16, 4); else NU_BY(__nv_bfloat16, 1); }
+#undef NU_BY
+#undef NU_GO
+  return mlxb_check_launch("norm_update");
 }

@@ -12,7 +12,9 @@
 //   by its root mean square over its dk columns after the rotation (no weight, `head_eps` >= 0); the values may have
 //   fewer heads than the keys (Hv of them, [n_pages, Hv, page, Dvr]: several key heads then read one value head); every value head may be
 //   divided by its root mean square over its dv columns (no weight, `v_eps` >= 0) before it enters the page; q may
-//   leave in float32 whatever the activation dtype is (for attention kernels that take float32 queries).
+//   leave in float32 whatever the activation dtype is (for attention kernels that take float32 queries), with a rounded
+//   copy beside it (`q16`).  The values may be mixed with those of an earlier layer (rows of Hv*dv columns in a buffer):
+//   (1 - lambda) v + lambda v_first goes into the page; the layer they come from leaves its own there (`v_keep`).
 // Norm, angle, sine and cosine are float32 (the angle is the float32 product of the position and a
 // float32 frequency, reduced accurately by sincosf).
 #include "common.cuh"
@@ -27,7 +29,8 @@ __global__ void qkv_prepare_kernel(const T* proj, int ld, int q_off, int k_off, 
                                    const int* __restrict__ block_table, int max_pages, int n_pages, int page,
                                    TQ* __restrict__ q_out, int ldq, T* __restrict__ k_pool, T* __restrict__ v_pool,
                                    int write, int* __restrict__ status, int interleaved, float v_eps, int Dvr, int Hv,
-                                   float mscale, float head_eps) {
+                                   float mscale, float head_eps, __nv_bfloat16* __restrict__ q16, int ldq16,
+                                   const T* v_first, T* v_keep, int ldvf, float lambda) {
   __shared__ float red[33];
   const int t = blockIdx.x;
   const int r = token_req[t];
@@ -52,6 +55,7 @@ __global__ void qkv_prepare_kernel(const T* proj, int ld, int q_off, int k_off, 
   pdl_wait();
   pdl_trigger();
   proj = after_wait(proj);
+  v_first = after_wait(v_first);
   const T* row = proj + (size_t)t * ld;
   float rq = 1.f, rk = 1.f;
   if (wq) {
@@ -95,8 +99,10 @@ __global__ void qkv_prepare_kernel(const T* proj, int ld, int q_off, int k_off, 
       const float rinv = 1.f / sqrtf(warp_sum(ss) / (float)dk + head_eps);
       for (int i = lane; i < Dh; i += 32) {
         const float a = i < dk ? value(i) * rinv : 0.f;
-        if (is_q) q_out[(size_t)t * ldq + (size_t)h * Dh + i] = from_f<TQ>(a);
-        else k_pool[(size_t)(slot + (long long)h * page) * Dh + i] = from_f<T>(a);
+        if (is_q) {
+          q_out[(size_t)t * ldq + (size_t)h * Dh + i] = from_f<TQ>(a);
+          if (q16) q16[(size_t)t * ldq16 + (size_t)h * Dh + i] = __float2bfloat16_rn(a);
+        } else k_pool[(size_t)(slot + (long long)h * page) * Dh + i] = from_f<T>(a);
       }
     }
   }
@@ -139,11 +145,18 @@ __global__ void qkv_prepare_kernel(const T* proj, int ld, int q_off, int k_off, 
     if (is_q) {
       dq[i] = from_f<TQ>(a);
       if (j >= 0) dq[j] = from_f<TQ>(b);
+      if (q16) {
+        __nv_bfloat16* dr = q16 + (size_t)t * ldq16 + (size_t)h * Dh;
+        dr[i] = __float2bfloat16_rn(a);
+        if (j >= 0) dr[j] = __float2bfloat16_rn(b);
+      }
     } else {
       dk_[i] = from_f<T>(a);
       if (j >= 0) dk_[j] = from_f<T>(b);
     }
   }
+  if (v_keep)
+    for (int e = threadIdx.x; e < Hv * dv; e += blockDim.x) v_keep[(size_t)t * ldvf + e] = row[v_off + e];
   if (slot >= 0 && v_eps >= 0.f) {
     // every value head divided by its root mean square: a warp a head
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
@@ -157,7 +170,9 @@ __global__ void qkv_prepare_kernel(const T* proj, int ld, int q_off, int k_off, 
   } else if (slot >= 0) {
     for (int e = threadIdx.x; e < Hv * Dvr; e += blockDim.x) {
       const int h = e / Dvr, i = e - h * Dvr;
-      v_pool[(size_t)(vslot + (long long)h * page) * Dvr + i] = i < dv ? row[v_off + h * dv + i] : from_f<T>(0.f);
+      T v = i < dv ? row[v_off + h * dv + i] : from_f<T>(0.f);
+      if (v_first && i < dv) v = from_f<T>((1.f - lambda) * to_f(v) + lambda * to_f(v_first[(size_t)t * ldvf + h * dv + i]));
+      v_pool[(size_t)(vslot + (long long)h * page) * Dvr + i] = v;
     }
   }
 }
@@ -165,18 +180,22 @@ __global__ void qkv_prepare_kernel(const T* proj, int ld, int q_off, int k_off, 
 // proj: [n_tokens, ...] at row stride ld holding q (Hq*dk columns from q_off), k (Hkv*dk from k_off) and v (Hkv*dv
 // from v_off); interleaved: pairs (2i, 2i+1) instead of (i, i+half); v_eps >= 0: value heads divided by their root mean
 // square with this eps; Hv: value heads (0: as many as key heads); mscale: factor on cosine and sine; head_eps >= 0: q and k
-// heads divided by their root mean square after the rotation; q_f32: q_out is float32 whatever dtype says; wq / wk: float32 norm weights over the whole q / k projection, or null for no norm; freq: float32
+// heads divided by their root mean square after the rotation; q16: bfloat16 copy of q_out at row stride ldq16, or null; v_first
+// (or null): [n_tokens, Hv*dv] at row stride ldvf, mixed into the values with weight lambda; v_keep (or null): the same rows
+// written from this projection's values; q_f32: q_out is float32 whatever dtype says; wq / wk: float32 norm weights over the whole q / k projection, or null for no norm; freq: float32
 // [half] rotation frequencies (half may be 0); k_pool [n_pages, Hkv, page, Dh], v_pool [n_pages, Hkv, page, Dvr]; q_out [n_tokens, Hq*Dh] at row stride ldq.
 MLXB_EXPORT int mlxb_qkv_prepare(int dtype, const void* proj, int ld, int q_off, int k_off, int v_off, int Hq, int Hkv,
                                  int dk, int dv, int Dh, const float* wq, const float* wk, float eps, const float* freq,
                                  int half, const int* positions, const int* token_req, const int* block_table,
                                  int max_pages, int n_pages, int page, void* q_out, int ldq, void* k_pool, void* v_pool,
                                  int write, int n_tokens, int* status, int interleaved, float v_eps, int q_f32, int Dvr,
-                                 int Hv, float mscale, float head_eps, cudaStream_t stream) {
+                                 int Hv, float mscale, float head_eps, void* q16, int ldq16, const void* v_first,
+                                 void* v_keep, int ldvf, float lambda, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (Hv <= 0) Hv = Hkv;
   if (Hq <= 0 || Hkv <= 0 || dk <= 0 || dv <= 0 || Dh < dk || Dvr < dv || 2 * half > dk || half < 0 || page <= 0 ||
-      (half > 0 && freq == nullptr) || ldq < Hq * Dh)
+      (half > 0 && freq == nullptr) || ldq < Hq * Dh || (q16 && ldq16 < Hq * Dh) || ((v_first || v_keep) && ldvf < Hv * dv) ||
+      (v_first && v_eps >= 0.f))
     return mlxb_fail(MLXB_BAD_ARG, "qkv_prepare: %d/%d heads, sizes %d/%d in %d, %d rotated pairs, page %d", Hq, Hkv, dk,
                      dv, Dh, half, page);
   const int work = (Hq + Hkv) * Dh;
@@ -184,7 +203,8 @@ MLXB_EXPORT int mlxb_qkv_prepare(int dtype, const void* proj, int ld, int q_off,
 #define QKVP_GO(T, TQ)                                                                                                  \
   launch_pdl(qkv_prepare_kernel<T, TQ>, dim3(n_tokens), dim3(threads), 0, stream, (const T*)proj, ld, q_off, k_off, v_off, \
              Hq, Hkv, dk, dv, Dh, wq, wk, eps, freq, half, positions, token_req, block_table, max_pages, n_pages, page,  \
-             (TQ*)q_out, ldq, (T*)k_pool, (T*)v_pool, write, status, interleaved, v_eps, Dvr, Hv, mscale, head_eps)
+             (TQ*)q_out, ldq, (T*)k_pool, (T*)v_pool, write, status, interleaved, v_eps, Dvr, Hv, mscale, head_eps, \
+             (__nv_bfloat16*)q16, ldq16, (const T*)v_first, (T*)v_keep, ldvf, lambda)
   if (dtype == MLXB_F32) QKVP_GO(float, float);
   else if (dtype == MLXB_BF16 && q_f32) QKVP_GO(__nv_bfloat16, float);
   else if (dtype == MLXB_BF16) QKVP_GO(__nv_bfloat16, __nv_bfloat16);

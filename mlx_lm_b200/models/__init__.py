@@ -1,2 +1,2 @@
 """Architectures that ship with the package; importing this package registers them."""
-from . import dalorax, gpt2, lelatar, nufetar, vobusun, zuluvik  # noqa: F401
+from . import dalorax, fisesun, gpt2, lelatar, nufetar, vobusun, zuluvik  # noqa: F401

@@ -855,6 +855,29 @@ def residual_update(x, y1, stream, w1=None, y2=None, w2=None, scale: float = 1.0
           _p(w2), ldy, float(scale), float(eps), _p(cast_out), ldc, R, D, stream)
 
 
+def norm_update(x, y1, weight, eps: float, stream, terms: int = 1, scale: float = 1.0, y2=None, token_req=None,
+                cast_out=None) -> None:
+    """In place on float32 rows: ``x[t] += rmsnorm(y) * weight`` with ``y = scale * sum_k y1[t * terms + k] + y2[t]``
+    (``y2``: float32 rows or None).  ``cast_out``: a copy of the new rows in its own dtype.  Rows whose ``token_req`` is
+    negative are left alone."""
+    _need(x, torch.float32, "norm_update x")
+    _need(y1, torch.float32, "norm_update y1")
+    _need(weight, torch.float32, "norm_update weight")
+    T, D = x.shape
+    if y1.shape != (T * terms, D) or weight.numel() != D or (y2 is not None and y2.shape != (T, D)):
+        raise KernelError(f"norm_update: x {tuple(x.shape)}, y1 {tuple(y1.shape)} of {terms} term(s), weight of {weight.numel()}")
+    if y2 is not None:
+        _need(y2, torch.float32, "norm_update y2")
+    if cast_out is not None and cast_out.shape != x.shape:
+        raise KernelError("norm_update: cast_out must have the shape of x")
+    _call("rms", "mlxb_norm_update", [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
+                                      c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+          dtype_code(cast_out.dtype) if cast_out is not None else F32, _p(x), _rows(x, "norm_update x"), _p(y1),
+          _rows(y1, "norm_update y1"), int(terms), float(scale), _p(y2), _rows(y2, "norm_update y2") if y2 is not None else 0,
+          _p(weight), float(eps), _p(token_req), _p(cast_out),
+          _rows(cast_out, "norm_update cast_out") if cast_out is not None else 0, T, D, stream)
+
+
 def head_difference(a, rep: int, value_dim: int, lam: float, eps: float, post: float, out, stream, token_req=None) -> None:
     """Two score maps over the same values combined per head: ``o = a1 - lam * a2``, divided by its root mean square
     over the head's ``value_dim`` columns (eps inside the root, no weight), times ``post``.  ``a``: float32
@@ -1121,17 +1144,160 @@ def rglru_scan(gates, r_bias, i_bias, decay, u, y, state, slots, token_req, req_
 
 
 # --------------------------------------------------------------------------
+# matrix memory with exponential gates (csrc/mlstm.cu)
+
+MLSTM_TILE = 128      # rows of a tile of mlstm_chunks at most
+
+
+def mlstm_gates(raw, f_off: int, cap: float, m_state, slots, token_req, req_first_token, coef, n_heads: int, stream,
+                tiled: bool = False, tile_rows: int = 0) -> None:
+    """Along every request's run of rows: ``i = cap tanh(z_i / cap)``, ``f = logsigmoid(cap tanh(z_f / cap))``,
+    ``m <- max(f + m, i)``, and the four numbers a row and head that ``mlstm_scan`` (``tiled`` False, and runs of one row) or
+    ``mlstm_chunks`` (``tiled``: runs of several rows, in tiles of ``tile_rows``) go by, into ``coef`` (float32 ``[T * heads *
+    4]``).  ``raw``: float32 ``[T, .]``, the input gates in columns 0.., the forget gates from ``f_off``; ``m_state`` float32
+    ``[slots, heads]``."""
+    _need(raw, torch.float32, "mlstm_gates raw")
+    _need(m_state, torch.float32, "mlstm_gates state")
+    _need(coef, torch.float32, "mlstm_gates coef")
+    T = raw.shape[0]
+    if m_state.shape[1:] != (n_heads,) or not m_state.is_contiguous() or coef.numel() < 4 * T * n_heads:
+        raise KernelError(f"mlstm_gates: state {tuple(m_state.shape)} for {n_heads} heads, coef of {coef.numel()} for {T} rows")
+    _call("mlstm", "mlxb_mlstm_gates", [c_void_p, c_int, c_int, c_float] + [c_void_p] * 5 + [c_int] * 4 + [c_void_p],
+          _p(raw), _rows(raw, "mlstm_gates raw"), int(f_off), float(cap), _p(m_state), _p(slots), _p(token_req),
+          _p(req_first_token), _p(coef), n_heads, int(tile_rows or PREFILL_TILE), int(bool(tiled)), slots.numel(), stream)
+
+
+def mlstm_gates_single(x, w, bias, cap: float, m_state, slots, token_req, req_first_token, coef, n_heads: int, stream) -> None:
+    """``mlstm_gates`` with the gates' projections in it, ``z = x w^T + bias`` (``w`` ``[2 heads, width]``, the input gates'
+    rows first; ``bias`` float32), for steps in which no request brings more than one row."""
+    _need(x, w.dtype, "mlstm_gates x")
+    _need(bias, torch.float32, "mlstm_gates bias")
+    _need(m_state, torch.float32, "mlstm_gates state")
+    _need(coef, torch.float32, "mlstm_gates coef")
+    T, D = x.shape
+    if (w.shape != (2 * n_heads, D) or not w.is_contiguous() or bias.numel() != 2 * n_heads or m_state.shape[1:] != (n_heads,)
+            or not m_state.is_contiguous() or coef.numel() < 4 * T * n_heads):
+        raise KernelError(f"mlstm_gates: w {tuple(w.shape)}, state {tuple(m_state.shape)} for {n_heads} heads and rows of {D}")
+    _call("mlstm", "mlxb_mlstm_gates_single", [c_int, c_void_p, c_int, c_void_p, c_void_p, c_float] + [c_void_p] * 5 + [c_int] * 4
+          + [c_void_p],
+          dtype_code(x.dtype), _p(x), _rows(x, "mlstm_gates x"), _p(w), _p(bias), float(cap), _p(m_state), _p(slots),
+          _p(token_req), _p(req_first_token), _p(coef), n_heads, D, slots.numel(), T, stream)
+
+
+def _mlstm_state(state, n_heads: int, what: str):
+    _need(state, torch.float32, what + " state")
+    _, H, V1, K = state.shape
+    if H != n_heads or V1 < 2 or not state.is_contiguous():
+        raise KernelError(f"{what}: state {tuple(state.shape)} for {n_heads} heads")
+    return H, K, V1 - 1
+
+
+def mlstm_scan(qkv, q_off: int, k_off: int, v_off: int, qscale: float, coef, state, slots, token_req, req_first_token, o, den,
+               n_heads: int, stream, max_run: int = 0) -> None:
+    """Per (request, head), token by token: ``S <- c0 S + c1 k v^T``, ``o = S^T (qscale q)`` with the row's first two numbers of
+    ``coef``.  ``qkv [T, .]`` holds q, k, v from the given column offsets; ``state`` float32 ``[slots, heads, V + 1, K]`` (a
+    head's state column by column; the last column takes 1 for v); ``o`` float32 ``[T, heads*V]``, not divided; ``den`` float32
+    ``[T * heads]``: the last column's result.  ``max_run`` > 0: requests that bring more rows are passed over."""
+    H, K, V = _mlstm_state(state, n_heads, "mlstm_scan")
+    for t, what in ((o, "o"), (den, "den"), (coef, "coef")):
+        _need(t, torch.float32, "mlstm_scan " + what)
+    T = qkv.shape[0]
+    if o.shape != (T, H * V) or den.numel() < T * H or coef.numel() < 4 * T * H:
+        raise KernelError(f"mlstm_scan: o {tuple(o.shape)} for {H} heads of {V} columns, {T} rows")
+    _call("mlstm", "mlxb_mlstm_scan", [c_int, c_void_p, c_int, c_int, c_int, c_int, c_float] + [c_void_p] * 6 + [c_int, c_void_p]
+          + [c_int] * 5 + [c_void_p],
+          dtype_code(qkv.dtype), _p(qkv), _rows(qkv, "mlstm_scan qkv"), q_off, k_off, v_off, float(qscale), _p(coef), _p(state),
+          _p(slots), _p(token_req), _p(req_first_token), _p(o), _rows(o, "mlstm_scan o"), _p(den), H, K, V, slots.numel(),
+          int(max_run), stream)
+
+
+def mlstm_chunks_supported(dtype, dim: int, tile_rows: int = 0) -> bool:
+    """Whether runs of several rows go through ``mlstm_chunks`` (bfloat16, heads of up to 256 key columns)."""
+    return dtype == torch.bfloat16 and 1 <= dim <= 256 and (tile_rows or PREFILL_TILE) <= MLSTM_TILE
+
+
+def mlstm_chunks_gated(dim: int, vdim: int) -> bool:
+    """Whether ``mlstm_chunks`` can finish a head's rows itself (one thread block has all columns of the head)."""
+    return vdim <= (128 if dim <= 128 else 64)
+
+
+def mlstm_chunks_scratch(n_tokens: int, n_requests: int, n_heads: int, dim: int, vdim: int, tile_rows: int = 0) -> int:
+    """Floats of scratch memory ``mlstm_chunks`` needs: a state per tile of a run."""
+    return (n_tokens // (tile_rows or PREFILL_TILE) + n_requests + 1) * n_heads * dim * (vdim + 1)
+
+
+def mlstm_chunks(qkv, q_off: int, k_off: int, v_off: int, qscale: float, coef, state, slots, token_req, req_first_token,
+                 req_first_position, tiles, n_tiles: int, scratch, n_heads: int, stream, out=None, den=None, gate=None,
+                 weight=None, gated=None, eps: float = 0.0, tile_rows: int = 0) -> None:
+    """``mlstm_scan`` for the requests that bring several rows, in tiles on tensor cores (bfloat16; three launches): a tile's
+    contribution to the state, the states along each run, the tiles' outputs.  ``coef``: the tiled numbers; ``tiles``: int32
+    ``[n_tiles, 4]`` = (first token row, rows, request, first position), at most ``tile_rows`` rows each.  ``out`` and ``den`` as
+    ``mlstm_scan``'s ``o`` and ``den``; or ``gate``, ``weight`` and ``gated`` (heads that ``mlstm_chunks_gated`` takes): what
+    ``mlstm_finish`` makes of them."""
+    _need(qkv, torch.bfloat16, "mlstm_chunks qkv")
+    H, K, V = _mlstm_state(state, n_heads, "mlstm_chunks")
+    _need(tiles, torch.int32, "mlstm_chunks tiles")
+    _need(scratch, torch.float32, "mlstm_chunks scratch")
+    _need(coef, torch.float32, "mlstm_chunks coef")
+    T, tile_rows = qkv.shape[0], tile_rows or PREFILL_TILE
+    if (tiles.numel() < 4 * n_tiles or coef.numel() < 4 * T * H
+            or scratch.numel() < mlstm_chunks_scratch(T, slots.numel(), H, K, V, tile_rows)):
+        raise KernelError(f"mlstm_chunks: state {tuple(state.shape)}, {n_tiles} tiles, scratch of {scratch.numel()}")
+    if not ((out is None) == (den is None) and (gate is None) == (gated is None) == (weight is None) and (out is None) != (gate is None)):
+        raise KernelError("mlstm_chunks: either out and den, or gate, weight and gated")
+    for t, dt in ((out, torch.float32), (gate, torch.bfloat16), (gated, torch.bfloat16)):
+        if t is not None:
+            _need(t, dt, "mlstm_chunks rows")
+            if t.shape != (T, H * V):
+                raise KernelError(f"mlstm_chunks: rows of {tuple(t.shape)} for {H} heads of {V}")
+    if weight is not None:
+        _need(weight, torch.float32, "mlstm_chunks weight")
+        if weight.numel() != H * V:
+            raise KernelError(f"mlstm_chunks: a weight of {weight.numel()} for {H} heads of {V}")
+    if den is not None:
+        _need(den, torch.float32, "mlstm_chunks den")
+        if den.numel() < T * H:
+            raise KernelError(f"mlstm_chunks: den of {den.numel()} for {T} rows of {H} heads")
+    rows = lambda t: 0 if t is None else _rows(t, "mlstm_chunks rows")
+    _call("mlstm", "mlxb_mlstm_chunks", [c_void_p, c_int, c_int, c_int, c_int, c_float] + [c_void_p] * 7 + [c_int, c_int, c_void_p]
+          + [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_float] + [c_int] * 4 + [c_void_p],
+          _p(qkv), _rows(qkv, "mlstm_chunks qkv"), q_off, k_off, v_off, float(qscale), _p(coef), _p(state), _p(slots),
+          _p(token_req), _p(req_first_token), _p(req_first_position), _p(tiles), int(n_tiles), int(tile_rows), _p(scratch),
+          _p(out), rows(out), _p(den), _p(gate), rows(gate), _p(weight), _p(gated), rows(gated), float(eps), H, K, V,
+          slots.numel(), stream)
+
+
+def mlstm_finish(o, den, coef, weight, gate, out, n_heads: int, eps: float, token_req, stream) -> None:
+    """``out = rms(o / (max(|den|, exp(-m)) + 1e-6)) * weight * sigmoid(gate)``, the root mean square over every head's columns
+    (``eps`` inside the root); ``exp(-m)`` is the last of a row's and head's four numbers in ``coef``.  Rows whose ``token_req``
+    is negative are left alone."""
+    for t, what in ((o, "o"), (den, "den"), (coef, "coef"), (weight, "weight")):
+        _need(t, torch.float32, "mlstm_finish " + what)
+    _need(gate, out.dtype, "mlstm_finish gate")
+    T, n = out.shape
+    if o.shape != (T, n) or gate.shape != (T, n) or weight.numel() != n or n % n_heads or den.numel() < T * n_heads \
+            or coef.numel() < 4 * T * n_heads:
+        raise KernelError(f"mlstm_finish: o {tuple(o.shape)}, gate {tuple(gate.shape)}, out {tuple(out.shape)}, {n_heads} heads")
+    _call("mlstm", "mlxb_mlstm_finish", [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float,
+                                         c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+          dtype_code(out.dtype), _p(o), _rows(o, "mlstm_finish o"), _p(den), _p(coef), _p(weight), _p(gate),
+          _rows(gate, "mlstm_finish gate"), _p(token_req), float(eps), _p(out), _rows(out, "mlstm_finish out"), n_heads,
+          n // n_heads, T, stream)
+
+
+# --------------------------------------------------------------------------
 # queries, keys and values into shape for the attention kernels (csrc/rotary.cu)
 
 _QKVP_ARGS = [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
               c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
-              c_void_p, c_int, c_int, c_void_p, c_int, c_float, c_int, c_int, c_int, c_float, c_float, c_void_p]
+              c_void_p, c_int, c_int, c_void_p, c_int, c_float, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int,
+              c_void_p, c_void_p, c_int, c_float, c_void_p]
 
 
 def qkv_prepare(proj, q_off: int, k_off: int, v_off: int, n_heads: int, n_kv_heads: int, dk: int, dv: int, q_norm,
                 k_norm, eps: float, freq, positions, token_req, block_table, k_pool, v_pool, q_out, write: bool, status,
                 stream, interleaved: bool = False, v_norm_eps: Optional[float] = None, mscale: float = 1.0,
-                head_norm_eps: Optional[float] = None) -> None:
+                head_norm_eps: Optional[float] = None, q_rounded=None, v_first=None, v_keep=None, v_lambda: float = 0.0) -> None:
     """From a fused projection ``proj [T, .]``: optional RMS norm over a token's whole q and whole k projection
     (float32 weights ``q_norm``, ``k_norm`` or None), rotation of the first ``2 * len(freq)`` dimensions of every
     head by the token's position (pairs ``(i, i + len(freq))``; ``freq`` float32 or None), q into ``q_out
@@ -1141,7 +1307,9 @@ def qkv_prepare(proj, q_off: int, k_off: int, v_off: int, n_heads: int, n_kv_hea
     factor on every cosine and sine (what a stretched rotation multiplies them with).  ``head_norm_eps``: every q and k
     head is divided by its root mean square over its ``dk`` columns AFTER the rotation (no weight).  ``v_pool`` may have
     fewer heads than ``k_pool`` (a divisor of them): the projection then holds that many value heads.  ``q_out`` may
-    be float32 in a bfloat16 run."""
+    be float32 in a bfloat16 run; ``q_rounded`` (bfloat16, as wide): a rounded copy of it.  ``v_first`` (the run's dtype, ``[T,
+    value heads * dv]``): the values that go into the page are ``(1 - v_lambda) v + v_lambda v_first``; ``v_keep`` (the same
+    shape): receives this projection's values as they are."""
     n_pages, Hkv, page, Dh = k_pool.shape
     _need(proj, k_pool.dtype, "qkv_prepare proj")
     if q_out.dtype != torch.float32:
@@ -1159,13 +1327,26 @@ def qkv_prepare(proj, q_off: int, k_off: int, v_off: int, n_heads: int, n_kv_hea
             _need(w, torch.float32, "qkv_prepare norm weight")
             if w.numel() != n:
                 raise KernelError(f"qkv_prepare: norm weight of {w.numel()} for {n} columns")
+    if q_rounded is not None:
+        _need(q_rounded, torch.bfloat16, "qkv_prepare q_rounded")
+        if q_rounded.shape[0] != proj.shape[0] or q_rounded.shape[1] < n_heads * Dh:
+            raise KernelError(f"qkv_prepare: q_rounded {tuple(q_rounded.shape)} for {n_heads} heads of {Dh}")
+    ldvf = 0
+    for t in (v_first, v_keep):
+        if t is not None:
+            _need(t, proj.dtype, "qkv_prepare values of another layer")
+            if t.shape != (proj.shape[0], Hv * dv) or (ldvf and _rows(t, "qkv_prepare values") != ldvf):
+                raise KernelError(f"qkv_prepare: values of another layer {tuple(t.shape)} for {Hv} heads of {dv}")
+            ldvf = _rows(t, "qkv_prepare values")
     _call("rotary", "mlxb_qkv_prepare", _QKVP_ARGS, dtype_code(k_pool.dtype), _p(proj), _rows(proj, "qkv_prepare proj"),
           q_off, k_off, v_off, n_heads, n_kv_heads, dk, dv, Dh, _p(q_norm), _p(k_norm), float(eps), _p(freq), half,
           _p(positions), _p(token_req), _p(block_table), block_table.shape[1], n_pages, page, _p(q_out),
           _rows(q_out, "qkv_prepare q_out"), _p(k_pool), _p(v_pool), int(bool(write)), proj.shape[0], _p(status),
           int(bool(interleaved)), -1.0 if v_norm_eps is None else float(v_norm_eps),
           int(q_out.dtype == torch.float32 and k_pool.dtype != torch.float32), v_pool.shape[3], Hv, float(mscale),
-          -1.0 if head_norm_eps is None else float(head_norm_eps), stream)
+          -1.0 if head_norm_eps is None else float(head_norm_eps), _p(q_rounded),
+          0 if q_rounded is None else _rows(q_rounded, "qkv_prepare q_rounded"), _p(v_first), _p(v_keep), ldvf, float(v_lambda),
+          stream)
 
 
 # --------------------------------------------------------------------------
@@ -1565,6 +1746,23 @@ def moe_plan(sel_expert, n_slots: int, n_experts: int, tile_rows: int, sorted_sl
           _p(sel_expert), n_slots, n_experts, tile_rows, max_tiles, _p(sorted_slots), _p(tile_info), _p(n_tiles), stream)
 
 
+def moe_plan_table(tokens, token_req, table, n_tokens: int, n_experts: int, tile_rows: int, sorted_slots, tile_info, n_tiles,
+                   status, stream) -> None:
+    """``moe_plan`` without a router: token ``t`` uses the experts in row ``tokens[t]`` of ``table`` (int32 ``[vocab, top]``);
+    slot ``t * top + c`` is its c-th.  Rows whose ``token_req`` is negative take no part; a token id outside the table sets a
+    bit in ``status``."""
+    for t, what in ((tokens, "tokens"), (table, "table"), (sorted_slots, "sorted"), (tile_info, "tile_info"), (n_tiles, "n_tiles")):
+        _need(t, torch.int32, "moe_plan_table " + what)
+    vocab, top = table.shape
+    n_slots = n_tokens * top
+    max_tiles = moe_max_tiles(n_slots, n_experts, tile_rows)
+    if not table.is_contiguous() or sorted_slots.numel() < n_slots or tile_info.numel() < 3 * max_tiles or tokens.numel() < n_tokens:
+        raise KernelError(f"moe_plan_table: {n_tokens} tokens, table {tuple(table.shape)}, {n_experts} experts")
+    _call("moe", "mlxb_moe_plan_table", [c_void_p] * 3 + [c_int] * 6 + [c_void_p] * 5,
+          _p(tokens), _p(token_req), _p(table), vocab, top, n_tokens, n_experts, tile_rows, max_tiles, _p(sorted_slots),
+          _p(tile_info), _p(n_tiles), _p(status), stream)
+
+
 GATED_UNITS = {"silu": 0, "bounded": 1}     # csrc/gated_unit.cuh
 
 
@@ -1572,7 +1770,7 @@ def moe_gemm(a, a_div: int, w, n_out: int, sorted_slots, tile_info, n_tiles, max
              sel_weight=None, gated: bool = False, unit: str = "silu", limit: float = 0.0) -> None:
     """``out[slot] = a[slot // a_div] @ w[expert(slot)].T`` for every slot of the plan; ``w [E, n_out, K]``.  ``gated``:
     ``w [E, 2 n_out, K]`` holds gate rows then up rows and the result is ``silu(s g) * (s u)`` with ``s`` the slot's
-    routing weight; with ``unit="bounded"`` it is ``s g' sigmoid(1.702 g') (u' + 1)``, ``g' = min(g, limit)``,
+    routing weight (1 without ``sel_weight``); with ``unit="bounded"`` it is ``s g' sigmoid(1.702 g') (u' + 1)``, ``g' = min(g, limit)``,
     ``u' = clamp(u, -limit, limit)`` (the weight on the unit's output).  ``out``: ``a``'s dtype or float32,
     ``[n_slots, n_out]``."""
     _need(a, None, "moe_gemm a")
@@ -1582,7 +1780,7 @@ def moe_gemm(a, a_div: int, w, n_out: int, sorted_slots, tile_info, n_tiles, max
         raise KernelError(f"moe_gemm: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
     if out.dtype not in (a.dtype, torch.float32):
         raise KernelError(f"moe_gemm: out {out.dtype} for inputs {a.dtype}")
-    if gated:
+    if gated and sel_weight is not None:
         _need(sel_weight, torch.float32, "moe_gemm sel_weight")
     _call("moe", "mlxb_moe_gemm", [c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, ctypes.c_longlong, c_int, c_int,
                                    c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float,
@@ -1626,7 +1824,7 @@ def moe_gemm_tc05(a, w, n_out: int, sorted_slots, tile_info, n_tiles, max_tiles:
     E, NW, K = w.shape
     if NW != (2 if gated else 1) * n_out or a.shape[1] != K or out.shape[1] != n_out or not w.is_contiguous():
         raise KernelError(f"moe_gemm_tc05: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
-    if gated:
+    if gated and sel_weight is not None:
         _need(sel_weight, torch.float32, "moe_gemm_tc05 sel_weight")
     _call("moe_tcgen05", "mlxb_moe_gemm_tc05", [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
                                                 c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_float,
@@ -1661,6 +1859,14 @@ def gated_unit(x, out, stream, unit: str = "silu", limit: float = 0.0) -> None:
     _call("elementwise", "mlxb_gated_unit", [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p],
           dtype_code(out.dtype), _p(x), _rows(x, "gated_unit x"), _p(out), _rows(out, "gated_unit out"), F_, T,
           GATED_UNITS[unit], float(limit), stream)
+
+
+def soft_cap(x, cap: float, stream) -> None:
+    """``x <- cap * tanh(x / cap)`` in place on a contiguous float32 tensor."""
+    _need(x, torch.float32, "soft_cap x")
+    if not x.is_contiguous():
+        raise KernelError(f"soft_cap: strides {x.stride()}")
+    _call("elementwise", "mlxb_soft_cap", [c_void_p, ctypes.c_longlong, c_float, c_void_p], _p(x), x.numel(), float(cap), stream)
 
 
 def scale_by_rows(x, index, table, first: int, out, status, stream) -> None:

@@ -15,7 +15,8 @@ Kinds of parts and the interface each must have
 ``Mixer``           ``cache_spec()`` (what it keeps per request: a
                     ``PagedKVSpec``, a ``StateSpec`` or None) and
                     ``forward(ctx, x, residual, cache) -> residual + mix(x)``
-``FeedForward``     ``forward(ctx, x, residual) -> residual + f(x)``
+``FeedForward``     ``forward(ctx, x, residual) -> residual + f(x)``; for blocks that
+                    norm the result before they add it, ``summands(ctx, x)``
 ``Block``           ``forward(ctx, x, cache) -> x'``: the arrangement of two
                     norms, a mixer and a feed-forward
 
@@ -41,6 +42,12 @@ class Init:
     """How the random-weights mode fills a tensor: normal(mean, std) or a constant."""
     mean: float = 0.0
     std: float = 0.02
+
+
+@dataclass(frozen=True)
+class RowChoice(Init):
+    """How the random-weights mode fills an integer table: every row holds different numbers out of ``0 .. n - 1``."""
+    n: int = 1
 
 
 @dataclass(frozen=True)
@@ -175,9 +182,22 @@ class Mixer(Part):
         raise NotImplementedError
 
 
+@dataclass
+class Summands:
+    """A sublayer's result as what has to be added up, all float32: ``scale * sum_k rows[t * terms + k] + extra[t]``."""
+    rows: torch.Tensor
+    terms: int = 1
+    scale: float = 1.0
+    extra: Optional[torch.Tensor] = None
+
+
 class FeedForward(Part):
     def fold_input_norm(self, norm: Norm) -> bool:
         return False
+
+    def summands(self, ctx, x) -> Summands:
+        rows, terms = self.branch(ctx, x)
+        return Summands(rows, terms)
 
     def forward(self, ctx, x, residual):
         raise NotImplementedError

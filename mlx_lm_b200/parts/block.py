@@ -11,7 +11,7 @@ from typing import Optional
 import torch
 
 from .. import ops
-from .base import VECTOR, Block, FeedForward, Init, Mixer, Norm, ParamSpec, register_part
+from .base import VECTOR, Block, FeedForward, Init, Mixer, Norm, ParamSpec, Summands, register_part
 
 # In bfloat16 a block lets its mixer and its feed-forward fold the norm before them into their first linear
 # layer (parts/linear.py, ``Linear.fold_norm``): steps of few rows then run no norm kernels inside the blocks.
@@ -263,6 +263,66 @@ class HyperBlock(Block):
         return x
 
 
+class OutputNormBlock(Block):
+    """A block over a float32 residual stream with a norm on every sublayer's result and none before it:
+    ``x += norm_1(mixer(x))``, then, if the layer has a feed-forward, ``x += norm_2(feed_forward(x))``.
+
+    The sublayers read the stream itself (in the run's dtype) and leave their results in float32 (``mixer.mix``,
+    ``feed_forward.summands``); one kernel adds a feed-forward's summands up, norms the sum (an RMS norm,
+    ``Norm.rms_args()``), adds it to the stream and leaves the new rows in the run's dtype for what reads them next: this
+    block's feed-forward, or the block that runs next (``ctx.next_block``), whose input then waits in ``ctx.carried``."""
+    replayable = True
+    kernel_libs = ("rms", "elementwise")
+
+    def __init__(self, norm_1: Norm, mixer: Mixer, norm_2: Optional[Norm] = None, feed_forward: Optional[FeedForward] = None):
+        if (norm_2 is None) != (feed_forward is None):
+            raise ValueError("a feed-forward and the norm on its result come together")
+        self.norm_1, self.mixer, self.norm_2, self.feed_forward = norm_1, mixer, norm_2, feed_forward
+
+    def children(self):
+        return tuple(p for p in (self.norm_1, self.mixer, self.norm_2, self.feed_forward) if p is not None)
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def _rows(self, ctx, x):
+        """The stream's rows in the run's dtype."""
+        if ctx.dtype == torch.float32:
+            return x
+        out = ctx.ws.get("stream_rows", *x.shape, ctx.dtype)
+        ops.label("stream.cast", 0.0, (4.0 + out.element_size()) * x.numel())
+        ops.join_rows(x, None, out, ctx.stream)
+        return out
+
+    def _update(self, ctx, x, y: Summands, norm: Norm, read_next: bool):
+        """``x += norm(y)``; the new rows in the run's dtype where something reads them next."""
+        T, D = x.shape
+        cast = ctx.ws.get("stream_rows", T, D, ctx.dtype) if read_next and ctx.dtype != torch.float32 else None
+        weight, eps = norm.rms_args()
+        ops.label(norm.name, (6.0 + y.terms) * T * D, (8.0 + 4.0 * y.terms + (4.0 if y.extra is not None else 0.0)
+                                                       + (cast.element_size() if cast is not None else 0.0)) * T * D)
+        ops.norm_update(x, y.rows, weight, eps, ctx.stream, terms=y.terms, scale=y.scale, y2=y.extra, token_req=ctx.token_req,
+                        cast_out=cast)
+        return x if cast is None else cast
+
+    def forward(self, ctx, x, cache):
+        carried, ctx.carried = getattr(ctx, "carried", None), None
+        h = carried[1] if carried is not None and carried[0] is self else self._rows(ctx, x)
+        nxt = getattr(ctx, "next_block", None)
+        if not isinstance(nxt, OutputNormBlock):
+            nxt = None
+        y = Summands(self.mixer.mix(ctx, h, cache))
+        if self.feed_forward is None:
+            h = self._update(ctx, x, y, self.norm_1, nxt is not None)
+        else:
+            h = self._update(ctx, x, y, self.norm_1, True)
+            h = self._update(ctx, x, self.feed_forward.summands(ctx, h), self.norm_2, nxt is not None)
+        if nxt is not None:
+            ctx.carried = (nxt, h)
+        return x
+
+
+register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "hyper", HyperBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "parallel", ParallelBlock)

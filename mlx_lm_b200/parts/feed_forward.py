@@ -5,7 +5,7 @@ epilogue and the residual add in the second's."""
 
 from __future__ import annotations
 
-from .base import VECTOR, FeedForward, Init, ParamSpec, register_part
+from .base import INT_TABLE, MATRIX, VECTOR, FeedForward, Init, ParamSpec, RowChoice, Summands, register_part
 import torch
 
 from .. import ops
@@ -102,6 +102,9 @@ class ExpertsMLP(FeedForward):
     -limit, limit)``, and the weight multiplies the unit's OUTPUT (``scale_input=False``).  ``shared``: a feed-forward
     that runs for every token beside the experts and is added.
 
+    ``table_vocab``: no router; an integer table ``<name>.table`` ``[table_vocab, top]`` names every token id's experts, each
+    with weight ``1 / top`` on its output (``summands`` hands that factor to the block's sum; the silu unit).
+
     The experts' weights are stacked at bind time (``[E, 2 inner, width]`` gate rows then up rows, ``[E, width,
     inner]``); a step routes (``ops.moe_route``), sorts its (token, choice) slots by expert into tiles
     (``ops.moe_plan``) and runs two products over the tiles, the gated unit in the first one's epilogue: ``ops.moe_gemm``
@@ -117,7 +120,8 @@ class ExpertsMLP(FeedForward):
                  expert_prefix: str = "e", gate_name: str = "gate", up_name: str = "up", down_name: str = "down",
                  init: Init = Init(), router_init: Init = Init(), correction: bool = False, groups=None, identity: int = 0,
                  renormalize_eps: float = 0.0, weight_scale: float = 1.0, unit: str = "silu", limit: float = 0.0,
-                 shared: FeedForward = None, correction_name: str = "correction"):
+                 shared: FeedForward = None, correction_name: str = "correction", table_vocab: int = 0,
+                 table_name: str = "table"):
         n_outputs = n_experts + int(identity)
         if n_experts < 0 or identity < 0 or not 1 <= top <= n_outputs:
             raise ValueError(f"{name}: {top} of {n_experts} experts and {identity} identity experts")
@@ -125,7 +129,9 @@ class ExpertsMLP(FeedForward):
             raise ValueError(f"{name}: router score {score!r} is not one of {sorted(ops.MOE_SCORES)}")
         if unit not in ops.GATED_UNITS:
             raise ValueError(f"{name}: gated unit {unit!r} is not one of {sorted(ops.GATED_UNITS)}")
-        if scale_input != (unit == "silu"):
+        if table_vocab and (identity or groups or correction or unit != "silu"):
+            raise ValueError(f"{name}: a table of experts has no router whose options could be set, and goes with the silu unit")
+        if not table_vocab and scale_input != (unit == "silu"):
             raise ValueError(f"{name}: the routing weight goes on the input of the silu unit and on the output of the "
                              f"bounded one; other pairings are not built")
         count, keep = (int(groups[0]), int(groups[1])) if groups else (1, 1)
@@ -138,18 +144,22 @@ class ExpertsMLP(FeedForward):
         self.shared = shared
         self.correction_name = f"{name}.{correction_name}" if correction else None
         self.correction = None
-        self.router = Linear(f"{name}.{router_name}", width, n_outputs, bias=False, weight_suffix="", init=router_init)
+        self.table_name, self.table_vocab, self.table = f"{name}.{table_name}", int(table_vocab), None
+        self.router = None
+        if not table_vocab:
+            self.router = Linear(f"{name}.{router_name}", width, n_outputs, bias=False, weight_suffix="", init=router_init)
         self.names = [(f"{name}.{expert_prefix}{e}.{gate_name}", f"{name}.{expert_prefix}{e}.{up_name}",
                        f"{name}.{expert_prefix}{e}.{down_name}") for e in range(n_experts)]
         self.init = init
         self.w_in = self.w_out = None
 
     def children(self):
-        return (self.router,) + ((self.shared,) if self.shared is not None else ())
+        return tuple(p for p in (self.router, self.shared) if p is not None)
 
     def param_specs(self):
-        from .base import MATRIX
         specs = []
+        if self.table_vocab:
+            specs.append(ParamSpec(self.table_name, (self.table_vocab, self.top), INT_TABLE, RowChoice(n=self.n_experts)))
         if self.correction_name:
             specs.append(ParamSpec(self.correction_name, (self.n_outputs,), VECTOR, Init(0.0, 0.02)))
         for g, u, d in self.names:
@@ -160,29 +170,47 @@ class ExpertsMLP(FeedForward):
 
     def bind(self, tensors, dtype, device) -> None:
         self.correction = tensors[self.correction_name].contiguous() if self.correction_name else None
+        if self.table_vocab:
+            self.table = tensors[self.table_name]
+            if self.table.numel() and not 0 <= int(self.table.min()) <= int(self.table.max()) < self.n_experts:
+                raise ValueError(f"{self.table_name}: an expert outside 0 .. {self.n_experts - 1}")
         if not self.names:        # identity experts only
             return
         self.w_in = torch.stack([torch.cat([tensors[g], tensors[u]], dim=0) for g, u, _ in self.names]).contiguous()
         self.w_out = torch.stack([tensors[d] for _, _, d in self.names]).contiguous()
 
     def branch(self, ctx, x):
-        if self.identity or self.shared is not None:
-            raise ops.KernelError(f"{self.name}: identity experts and a shared expert add to the stream themselves (forward)")
+        if self.identity or self.shared is not None or self.table_vocab:
+            raise ops.KernelError(f"{self.name}: identity experts and a shared expert add to the stream themselves (forward); "
+                                  f"experts out of a table come with a factor (summands)")
         y, _, _ = self._experts(ctx, x)
         return y, self.top
+
+    def summands(self, ctx, x):
+        if self.identity:
+            raise ops.KernelError(f"{self.name}: identity experts add to the stream themselves (forward)")
+        y, _, _ = self._experts(ctx, x)
+        extra = None
+        if self.shared is not None:
+            extra, terms = self.shared.branch(ctx, x)
+            if terms != 1:
+                raise ops.KernelError(f"{self.name}: a shared expert that leaves {terms} rows a token")
+        return Summands(y, self.top, 1.0 / self.top if self.table_vocab else 1.0, extra)
 
     def _experts(self, ctx, x):
         """The chosen experts' rows, float32 ``[T * top, width]`` (rows of identity experts are not written), with the
         choices ``sel_expert`` and their weights."""
         T, E, top, F_, D = x.shape[0], self.n_experts, self.top, self.inner, self.width
         S, EO = T * top, self.n_outputs
-        logits = self.router.forward(ctx, x, ctx.ws.get("moe_logits", T, (EO + 7) // 8 * 8, torch.float32)[:, :EO])
-        sel_e = ctx.ws.flat("moe_sel_expert", S, torch.int32)
-        sel_w = ctx.ws.flat("moe_sel_weight", S, torch.float32)
-        ops.label(self.name + ".route", 8.0 * T * EO, 4.0 * T * EO + 8.0 * S)
-        ops.moe_route(logits, ctx.token_req, top, sel_e, sel_w, ctx.stream, score=self.score, renormalize=self.renormalize,
-                      correction=self.correction, groups=self.groups, keep_groups=self.keep_groups, identity=self.identity,
-                      renormalize_eps=self.renormalize_eps, weight_scale=self.weight_scale)
+        sel_e = sel_w = None
+        if not self.table_vocab:
+            logits = self.router.forward(ctx, x, ctx.ws.get("moe_logits", T, (EO + 7) // 8 * 8, torch.float32)[:, :EO])
+            sel_e = ctx.ws.flat("moe_sel_expert", S, torch.int32)
+            sel_w = ctx.ws.flat("moe_sel_weight", S, torch.float32)
+            ops.label(self.name + ".route", 8.0 * T * EO, 4.0 * T * EO + 8.0 * S)
+            ops.moe_route(logits, ctx.token_req, top, sel_e, sel_w, ctx.stream, score=self.score, renormalize=self.renormalize,
+                          correction=self.correction, groups=self.groups, keep_groups=self.keep_groups, identity=self.identity,
+                          renormalize_eps=self.renormalize_eps, weight_scale=self.weight_scale)
         y = ctx.ws.get("moe_out", S, D, torch.float32)
         if E == 0:
             return y, sel_e, sel_w
@@ -198,7 +226,11 @@ class ExpertsMLP(FeedForward):
         order = ctx.ws.flat("moe_sorted", S, torch.int32)
         tiles = ctx.ws.flat("moe_tiles", 3 * max_tiles + 1, torch.int32)
         n_tiles = tiles[3 * max_tiles:]
-        ops.moe_plan(sel_e, S, E, rows, order, tiles, n_tiles, ctx.stream)
+        if self.table_vocab:
+            ops.label(self.name + ".plan", 0.0, 4.0 * T + 8.0 * S)
+            ops.moe_plan_table(ctx.tokens, ctx.token_req, self.table, T, E, rows, order, tiles, n_tiles, ctx.status, ctx.stream)
+        else:
+            ops.moe_plan(sel_e, S, E, rows, order, tiles, n_tiles, ctx.stream)
         h = ctx.ws.get("moe_hidden", S, F_, x.dtype)
         es = x.element_size()
         if many:
@@ -219,6 +251,8 @@ class ExpertsMLP(FeedForward):
         return y, sel_e, sel_w
 
     def forward(self, ctx, x, residual):
+        if self.table_vocab and self.top != 1:
+            raise ops.KernelError(f"{self.name}: experts out of a table come with a factor (summands)")
         y, sel_e, sel_w = self._experts(ctx, x)
         terms = self.top
         ops.label(self.name + ".sum", terms * x.shape[0] * self.width, 4.0 * (terms + 2) * x.shape[0] * self.width)

@@ -294,6 +294,11 @@ class TalkingHeadsAttention(Mixer):
     * ``softcap``: scores become ``softcap * tanh(score / softcap)`` after the scale, before the softmax;
     * ``keep_first``: beside the window, the first ``keep_first`` positions of the sequence stay visible to every later
       position (``j <= p and (p - j < window or j < keep_first)``); their pages are never given back;
+    * ``qk_norm``: an RMS norm over a token's whole q projection, and whole k projection, before the heads are split and
+      turned, with plain weights ``<name>.q.norm`` / ``<name>.k.norm`` (eps inside the root);
+    * ``value_mix``: values mixed with those of an earlier layer, ``v <- (1 - lambda) v + lambda v_first`` with one learned
+      number ``<name>.vmix``, before they enter the page.  The layer whose values the others take has ``"first"`` (its own
+      number is not used), the others ``"mix"``; ``v_first`` is the step's own rows, so nothing of it is kept beyond a step;
     * ``own_kv=False``: the layer has no key and value projections; it reads the pages another layer wrote (the run
       order points it there with ``write=False``) with its own queries, mask, scale and gate.  ``cache_window`` and
       ``cache_keep_first`` say what the shared pages must keep when the layers that read them differ in their masks
@@ -310,7 +315,13 @@ class TalkingHeadsAttention(Mixer):
                  chunk: Optional[int] = None, init: Init = Init(), bias_init: Init = Init(), column_gate: bool = False,
                  softcap: float = 0.0, keep_first: int = 0, own_kv: bool = True, cache_window: Optional[int] = None,
                  cache_keep_first: Optional[int] = None, rot_scaling: Optional[dict] = None, head_norm: bool = False,
-                 out_bias: Optional[bool] = None):
+                 out_bias: Optional[bool] = None, qk_norm: bool = False, value_mix: Optional[str] = None):
+        if value_mix not in (None, "first", "mix") or (value_mix and (value_norm or not own_kv)):
+            raise ValueError(f"{name}: value_mix {value_mix!r}: 'first' or 'mix', of the layer's own values without a norm")
+        if qk_norm and not own_kv:
+            raise ValueError(f"{name}: a layer that reads another layer's pages does not norm their keys")
+        self.qk_norm, self.value_mix, self.vmix = qk_norm, value_mix, 0.0
+        self.q_norm = self.k_norm = None
         if n_heads % n_kv_heads:
             raise ValueError(f"{name}: {n_heads} query heads are not a multiple of {n_kv_heads} key/value heads")
         if rot_dims % 2 or rot_dims > dim:
@@ -344,10 +355,10 @@ class TalkingHeadsAttention(Mixer):
         self.has_bias, self.bias_init = bias, bias_init
         self.has_out_bias = bias if out_bias is None else bool(out_bias)
         self.talk = self.freq = None
-        if dim == 64 and vdim == 64 and not talk and not chunk and not head_gate:
+        if dim == 64 and vdim % 64 == 0 and not talk and not chunk and not head_gate:
             # plain heads of 64: prompt portions run on the tcgen05 kernel (queries that were turned or normed reach it
             # through a bfloat16 copy)
-            self.kernel_libs = type(self).kernel_libs + ("attention_prefill_tc", "elementwise")
+            self.kernel_libs = type(self).kernel_libs + ("attention_prefill_tc",)
 
     def children(self):
         return (self.proj, self.out)
@@ -362,11 +373,20 @@ class TalkingHeadsAttention(Mixer):
             specs.append(ParamSpec(f"{self.name}.talk", (self.n_heads, self.n_heads), VECTOR, Init(0.0, 0.5)))
         if self.has_out_bias:
             specs.append(ParamSpec(f"{self.name}.o.b", (self.width,), VECTOR, self.bias_init))
+        if self.qk_norm:
+            specs += [ParamSpec(f"{self.name}.q.norm", (self.n_heads * self.dim,), VECTOR, Init(1.0, 0.1)),
+                      ParamSpec(f"{self.name}.k.norm", (self.n_kv_heads * self.dim,), VECTOR, Init(1.0, 0.1))]
+        if self.value_mix:
+            specs.append(ParamSpec(f"{self.name}.vmix", (), VECTOR, Init(0.5, 0.1)))
         return specs
 
     def bind(self, tensors, dtype, device) -> None:
         if self.has_talk:
             self.talk = tensors[f"{self.name}.talk"].contiguous()
+        if self.qk_norm:
+            self.q_norm, self.k_norm = tensors[f"{self.name}.q.norm"], tensors[f"{self.name}.k.norm"]
+        if self.value_mix == "mix":
+            self.vmix = float(tensors[f"{self.name}.vmix"])
         if self.rot_dims:
             f, self.rot_mscale = rotation_frequencies(self.rot_dims, self.rot_base, self.rot_scaling)
             self.freq = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(device)
@@ -393,15 +413,15 @@ class TalkingHeadsAttention(Mixer):
         self.proj.forward(ctx, x, proj)
         q = ctx.ws.get("attn_q32", T, H * self.key_row, torch.float32)
         ops.label(self.name + ".prepare", 8.0 * T * n, (x.element_size() + 4.0) * T * n)
-        self._prepare(ctx, proj, cache, q)
-        # without a rotation (and without a norm of the heads) the product's own (rounded) query columns are the queries
-        q_rounded = proj[:, :H * self.dim] if not self.rot_dims and not self.head_norm and proj.dtype == cache.k.dtype else None
+        # without a rotation (and without a norm of the queries) the product's own (rounded) query columns are the queries
+        plain_q = not self.rot_dims and not self.head_norm and not self.qk_norm
+        q_rounded = proj[:, :H * self.dim] if plain_q and proj.dtype == cache.k.dtype else None
+        copy = None
         if (q_rounded is None and ctx.n_portion and ctx.portion_tiles is not None and "attention_prefill_tc" in self.kernel_libs
                 and proj.dtype == torch.bfloat16 and cache.k.dtype == torch.bfloat16 and ops.PREFILL_TC):
             # turned or normed queries of plain heads of 64: the tcgen05 kernel for portions takes them in bfloat16
-            q_rounded = ctx.ws.get("attn_q16", T, H * self.key_row, torch.bfloat16)
-            ops.label(self.name + ".prepare.cast", 0.0, 6.0 * T * H * self.key_row)
-            ops.join_rows(q, None, q_rounded, ctx.stream)
+            q_rounded = copy = ctx.ws.get("attn_q16", T, H * self.key_row, torch.bfloat16)
+        self._prepare(ctx, proj, cache, q, copy)
         o = ctx.ws.get("attn_out", T, H * self.vdim, x.dtype)
         if ops.recording():
             pairs, keys = visible_pairs(ctx, self.window, self.chunk)
@@ -416,14 +436,18 @@ class TalkingHeadsAttention(Mixer):
                                 gate=gate, softcap=self.softcap, keep_first=self.keep_first, q_rounded=q_rounded)
         return o
 
-    def _prepare(self, ctx, proj, cache, q) -> None:
+    def _prepare(self, ctx, proj, cache, q, q_rounded=None) -> None:
         H, G = self.n_heads, self.n_kv_heads
+        mix = {}
+        if self.value_mix:
+            rows = ctx.ws.get("attn_v_first", proj.shape[0], G * self.vdim, proj.dtype)
+            mix = dict(v_keep=rows) if self.value_mix == "first" else dict(v_first=rows, v_lambda=self.vmix)
         # (a layer without key and value projections passes offsets that are never read: nothing is written)
-        ops.qkv_prepare(proj, 0, H * self.dim, (H + G) * self.dim, H, G, self.dim, self.vdim, None, None, self.eps,
+        ops.qkv_prepare(proj, 0, H * self.dim, (H + G) * self.dim, H, G, self.dim, self.vdim, self.q_norm, self.k_norm, self.eps,
                         self.freq, ctx.positions, ctx.token_req, cache.block_table, cache.k, cache.v, q, cache.write,
                         ctx.status, ctx.stream, interleaved=self.interleaved,
                         v_norm_eps=self.eps if self.value_norm else None, mscale=self.rot_mscale,
-                        head_norm_eps=self.eps if self.head_norm else None)
+                        head_norm_eps=self.eps if self.head_norm else None, q_rounded=q_rounded, **mix)
 
 
 class LatentAttention(Mixer):

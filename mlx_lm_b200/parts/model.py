@@ -118,12 +118,14 @@ class TokenPairEmbedding(Part):
 
 class OutputHead(Part):
     """Logits in float32.  Tied: the embedding table is the weight and there is no bias
-    (``wte.as_linear``, mlx_lm/models/gpt2.py:166-167); untied: a linear layer of its own."""
+    (``wte.as_linear``, mlx_lm/models/gpt2.py:166-167); untied: a linear layer of its own.  ``softcap``: the logits become
+    ``softcap * tanh(logits / softcap)``."""
     replayable = True
 
     def __init__(self, vocab_size: int, width: int, tied_to: Optional[TokenEmbedding] = None,
-                 name: str = "lm_head", bias: bool = False, weight_suffix: str = ".weight", init: Init = Init()):
-        self.vocab_size, self.width, self.tied_to = vocab_size, width, tied_to
+                 name: str = "lm_head", bias: bool = False, weight_suffix: str = ".weight", init: Init = Init(),
+                 softcap: float = 0.0):
+        self.vocab_size, self.width, self.tied_to, self.softcap = vocab_size, width, tied_to, float(softcap or 0.0)
         self.linear = Linear(name, width, vocab_size, bias=bias and tied_to is None, weight_suffix=weight_suffix,
                              init=init)
 
@@ -131,7 +133,7 @@ class OutputHead(Part):
         return () if self.tied_to is not None else (self.linear,)
 
     def all_kernel_libs(self):
-        return list(self.linear.kernel_libs)
+        return list(self.linear.kernel_libs) + (["elementwise"] if self.softcap else [])
 
     def bind(self, tensors, dtype, device) -> None:
         if self.tied_to is not None:
@@ -140,6 +142,9 @@ class OutputHead(Part):
     def forward(self, ctx, x):
         out = ctx.ws.get("logits", x.shape[0], self.vocab_size, torch.float32)
         out = self.linear.forward(ctx, x, out)
+        if self.softcap:
+            ops.label("head.softcap", 3.0 * out.numel(), 8.0 * out.numel())
+            ops.soft_cap(out, self.softcap, ctx.stream)
         ops.label("after the output head")
         return out
 

@@ -65,13 +65,29 @@ def rotation_frequencies(dims: int, base: float, scaling: Optional[dict] = None)
     ``d(t) = dims * ln(original / (2 pi t)) / (2 ln base)`` (the pair that makes ``t`` turns over ``original``
     positions), ``lo = max(floor(d(fast)), 0)``, ``hi = min(ceil(d(slow)), dims - 1)`` and
     ``ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)``, the frequency becomes
-    ``f_i / factor * ramp_i + f_i * (1 - ramp_i)`` and cosine and sine are multiplied by ``0.1 ln(factor) + 1``."""
+    ``f_i / factor * ramp_i + f_i * (1 - ramp_i)`` and cosine and sine are multiplied by ``0.1 ln(factor) + 1``.
+    A ``scaling`` with ``low`` and ``high`` instead goes by the wavelength ``l_i = 2 pi / f_i`` (the rule of Llama 3.1): ``f_i``
+    where ``l_i < original / high``, ``f_i / factor`` where ``l_i > original / low``, and between them
+    ``(1 - s) f_i / factor + s f_i`` with ``s = (original / l_i - low) / (high - low)``; cosine and sine as they are."""
     import math
 
     f = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
     if not scaling:
         return f, 1.0
     factor, original = float(scaling["factor"]), float(scaling["original"])
+    if "low" in scaling:
+        low, high = float(scaling["low"]), float(scaling["high"])
+        out = []
+        for fi in f:
+            turns = original * fi / (2.0 * math.pi)        # turns the pair makes over ``original`` positions
+            if turns > high:
+                out.append(fi)
+            elif turns < low:
+                out.append(fi / factor)
+            else:
+                s = (turns - low) / (high - low) if high != low else 1.0
+                out.append((1.0 - s) * fi / factor + s * fi)
+        return out, 1.0
 
     def pair_of(turns: float) -> float:
         return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))

@@ -1,6 +1,6 @@
 """Mixers that keep a state of fixed size per request instead of keys and values: the selective
-state-space layer of Mamba-2, the gated delta rule, RWKV's time mixing, retention and the real-gated linear
-recurrent unit.  Some read their inputs through short causal
+state-space layer of Mamba-2, the gated delta rule, RWKV's time mixing, retention, the matrix memory of xLSTM and the
+real-gated linear recurrent unit.  Some read their inputs through short causal
 convolutions whose last ``taps - 1`` inputs are part of the state.  State is float32 and lives in the
 cache manager's slots; a step reads it at the start of each request's run of tokens and writes it back
 at the end, so prompts may be cut into portions anywhere and decoding continues from it.
@@ -333,6 +333,94 @@ class RetentionMixer(Mixer):
         return self.out.forward(ctx, self._gated(ctx, x, cache), residual, residual=residual)
 
 
+class MLSTMMixer(Mixer):
+    """The matrix memory of xLSTM: linear attention with exponential gates and a denominator.  ``q``, ``k`` (``heads x dim``, q
+    times ``dim**-0.5``), ``v`` (``heads x vdim``); per head ``i = cap tanh((W_i x + b) / cap)`` (``<name>.i``, ``<name>.i.b``)
+    and ``f = logsigmoid(cap tanh((W_f x + b) / cap))``; with a running maximum ``m <- max(f + m, i)`` that starts at 0,
+    ``S <- exp(f + m_before - m) S + exp(i - m) k v^T``, ``n`` likewise with ``k`` alone,
+    ``o = S^T q / (max(|n . q|, exp(-m)) + 1e-6)``; every head's ``o`` is divided by its root mean square (eps inside the root),
+    times ``norm`` (one weight per column), times ``sigmoid(W_g x)``, then ``<name>.o``.  The gates' products are left in
+    float32; everything between the projections and the output gate is float32.
+
+    ``n`` is kept as one more column of the state (its v is 1), the maxima as a state of their own."""
+    replayable = True
+    kernel_libs = ("mlstm",)
+
+    def __init__(self, name: str, width: int, n_heads: int, dim: int, vdim: int, gate_cap: float, eps: float, init: Init = Init()):
+        if not 1 <= dim <= 512:
+            raise ValueError(f"{name}: heads of {dim} key columns (1 to 512)")
+        if not gate_cap > 0:
+            raise ValueError(f"{name}: gate_cap {gate_cap!r} must be positive")
+        self.name, self.width, self.n_heads, self.dim, self.vdim = name, width, n_heads, dim, vdim
+        self.gate_cap, self.eps = float(gate_cap), float(eps)
+        self.qk_width, self.v_width = n_heads * dim, n_heads * vdim
+        self.proj = FusedLinear(f"{name}.qkvg", width, [(f"{name}.q", self.qk_width), (f"{name}.k", self.qk_width),
+                                                        (f"{name}.v", self.v_width), (f"{name}.g", self.v_width)], init=init)
+        self.gates = FusedLinear(f"{name}.if", width, [(f"{name}.i", n_heads), (f"{name}.f", n_heads)], init=init,
+                                 biases={f"{name}.{g}": f"{name}.{g}.b" for g in "if"}, bias_init=Init(0.0, 1.0))
+        self.out = Linear(f"{name}.o", self.v_width, width, bias=False, weight_suffix="", init=Init(0.0, self.v_width ** -0.5))
+        self.norm_w = None
+
+    def children(self):
+        return (self.proj, self.gates, self.out)
+
+    def cache_spec(self):
+        return {"memory": StateSpec((self.n_heads, self.vdim + 1, self.dim)),      # column by column: the kernels' layout
+                "max": StateSpec((self.n_heads,))}
+
+    def param_specs(self) -> List[ParamSpec]:
+        return [ParamSpec(f"{self.name}.norm", (self.v_width,), VECTOR, Init(1.0, 0.1))]
+
+    def bind(self, tensors, dtype, device) -> None:
+        self.norm_w = tensors[f"{self.name}.norm"].contiguous()
+
+    def _gated(self, ctx, x, cache):
+        T, H, VW, es = x.shape[0], self.n_heads, self.v_width, x.element_size()
+        n = self.proj.n_out
+        proj = ctx.ws.get("mlstm_proj", T, (n + 7) // 8 * 8, x.dtype)[:, :n]
+        self.proj.forward(ctx, x, proj)
+        v_off = 2 * self.qk_width
+        gate = proj[:, v_off + VW:v_off + 2 * VW]
+        memory, maxima = cache.side("memory"), cache.side("max")
+        where = (memory.slots, ctx.token_req, ctx.req_first_token)
+        coef = ctx.ws.flat("mlstm_coef", 4 * T * H, torch.float32)
+        tiled = ctx.n_portion > 0 and ctx.portion_tiles is not None and ops.mlstm_chunks_supported(x.dtype, self.dim)
+        if ctx.n_portion == 0:       # a row a request: the gates' products and the maximum's step in one launch
+            ops.label(self.name + ".gates", 4.0 * T * H * self.width, es * (T + 2 * H) * self.width + 24.0 * T * H)
+            ops.mlstm_gates_single(x, self.gates.weight, self.gates.bias, self.gate_cap, maxima.state, *where, coef, H, ctx.stream)
+        else:
+            raw = ctx.ws.get("mlstm_raw", T, (2 * H + 7) // 8 * 8, torch.float32)[:, :2 * H]
+            self.gates.forward(ctx, x, raw)
+            ops.label(self.name + ".gates", 60.0 * T * H, 24.0 * T * H)
+            ops.mlstm_gates(raw, H, self.gate_cap, maxima.state, *where, coef, H, ctx.stream, tiled=tiled)
+        g = ctx.ws.get("mlstm_gated", T, (VW + 7) // 8 * 8, x.dtype)[:, :VW]
+        cost = (6.0 * T * (VW + H) * self.dim, es * T * (v_off + VW) + 16.0 * T * H + 8.0 * min(T, ctx.n_requests) * (VW + H) * self.dim)
+        fused = tiled and ctx.n_single == 0 and ops.mlstm_chunks_gated(self.dim, self.vdim)      # the tiles' own kernel finishes its rows
+        o = None if fused else ctx.ws.get("mlstm_o", T, VW, torch.float32)
+        den = None if fused else ctx.ws.flat("mlstm_den", T * H, torch.float32)
+        heads = (proj, 0, self.qk_width, v_off, self.dim ** -0.5, coef, memory.state)
+        if tiled:
+            scratch = ctx.ws.flat("mlstm_states", ops.mlstm_chunks_scratch(T, ctx.n_requests, H, self.dim, self.vdim), torch.float32)
+            ops.label(self.name + ".memory", cost[0], cost[1] + (2.0 * es if fused else 4.0) * T * VW)
+            ops.mlstm_chunks(*heads, *where, ctx.req_first_position, ctx.portion_tiles, ctx.n_portion_tiles, scratch, H, ctx.stream,
+                             **(dict(gate=gate, weight=self.norm_w, gated=g, eps=self.eps) if fused else dict(out=o, den=den)))
+            if fused:
+                return g
+        if not tiled or ctx.n_single:
+            ops.label(self.name + ".memory", cost[0], cost[1] + 4.0 * T * VW)
+            ops.mlstm_scan(*heads, *where, o, den, H, ctx.stream, max_run=1 if tiled else 0)
+        ops.label(self.name + ".norm", 10.0 * T * VW, (4.0 + 2 * es) * T * VW)
+        ops.mlstm_finish(o, den, coef, self.norm_w, gate, g, H, self.eps, ctx.token_req, ctx.stream)
+        return g
+
+    def mix(self, ctx, x, cache, tag: str = "mix_out"):
+        g = self._gated(ctx, x, cache)
+        return self.out.forward(ctx, g, ctx.ws.get(tag, x.shape[0], self.width, torch.float32))
+
+    def forward(self, ctx, x, residual, cache):
+        return self.out.forward(ctx, self._gated(ctx, x, cache), residual, residual=residual)
+
+
 class RGLRUMixer(Mixer):
     """A recurrent block of two branches of ``inner`` columns: ``y = gelu_tanh(W_y x + b)`` and ``u``, a short causal
     convolution with bias (``<name>.conv`` ``[inner, taps]``, ``<name>.conv.b``; no activation) of ``W_x x + b``, through a
@@ -412,6 +500,7 @@ class RGLRUMixer(Mixer):
         return self.out.forward(ctx, self._gated(ctx, x, cache), residual, residual=residual)
 
 
+register_part("mixer", "mlstm", MLSTMMixer)
 register_part("mixer", "retention", RetentionMixer)
 register_part("mixer", "rglru", RGLRUMixer)
 register_part("mixer", "mamba2", Mamba2Mixer)

@@ -24,7 +24,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..config import get_architecture, load_config
-from ..parts.base import INT_TABLE, MATRIX, VECTOR, ParamSpec
+from ..parts.base import INT_TABLE, MATRIX, VECTOR, ParamSpec, RowChoice
 from ..parts.model import Model, ModelDescription
 
 PREFIXES = ("transformer.", "model.")
@@ -142,12 +142,16 @@ def load_model(model_path: str, dtype="bfloat16", device="cuda", model_config: O
 def random_tensors(description: ModelDescription, seed: int, dtype: torch.dtype = torch.bfloat16
                    ) -> Dict[str, torch.Tensor]:
     """Every tensor of the model drawn in float32 on the CPU from one generator seeded with
-    ``seed``, in the fixed order of ``param_specs()``, then rounded to ``dtype``."""
+    ``seed``, in the fixed order of ``param_specs()``, then rounded to ``dtype`` (integer tables: int32)."""
     g = torch.Generator(device="cpu").manual_seed(int(seed))
     out: Dict[str, torch.Tensor] = {}
     for s in description.param_specs():
         if s.kind == INT_TABLE:
-            raise WeightError(f"{s.name}: the random-weights mode has no rule for integer tables")
+            if not isinstance(s.init, RowChoice) or len(s.shape) != 2:
+                raise WeightError(f"{s.name}: the random-weights mode has no rule for this integer table")
+            draws = torch.rand((s.shape[0], s.init.n), generator=g, dtype=torch.float32)
+            out[s.name] = draws.argsort(dim=1)[:, :s.shape[1]].to(torch.int32).contiguous()
+            continue
         if s.init.std == 0.0:
             t = torch.full(s.shape, float(s.init.mean), dtype=torch.float32)
         else:
