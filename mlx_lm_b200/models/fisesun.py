@@ -110,7 +110,7 @@ class ModelArgs(BaseModelArgs):
             _positive_int(where + ".expert.ff", mlp["expert"]["ff"])
             if not 1 <= mlp["router"]["top"] <= mlp["router"]["experts"]:
                 raise ConfigError(f"{where}.router: top {mlp['router']['top']} of {mlp['router']['experts']}")
-            if mlp.get("shared"):
+            if mlp.get("shared") is not None:
                 need_keys(mlp["shared"], ["ff"], where + ".shared")
                 _positive_int(where + ".shared.ff", mlp["shared"]["ff"])
         else:
@@ -139,7 +139,7 @@ def _feed_forward(name: str, D: int, mlp: dict, vocab: int):
     lin = Init(0.0, D ** -0.5)
     if mlp["kind"] == "dense":
         return GatedMLP(name, D, mlp["ff"], init=lin)
-    shared = GatedMLP(name + ".shared", D, mlp["shared"]["ff"], init=lin) if mlp.get("shared") else None
+    shared = GatedMLP(name + ".shared", D, mlp["shared"]["ff"], init=lin) if mlp.get("shared") is not None else None
     return ExpertsMLP(name, D, mlp["expert"]["ff"], mlp["router"]["experts"], mlp["router"]["top"], init=lin, shared=shared,
                       table_vocab=vocab)
 
