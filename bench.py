@@ -750,6 +750,39 @@ def vobusun_config(width, vocab):
             "embedding": {"scale": 8.0, "bigram": {"buckets": 4093, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
 
 
+def fisesun_config(width, vocab):
+    """Ten layers of the sizes a model of this width would have: six matrix memories with heads of 64 x 128; four layers of
+    attention with heads of 64 and a quarter as many key/value heads, a window of 1024 positions beside four kept first ones,
+    scores capped at 30, mixed values, rotations stretched by wavelength; feed-forwards in turn dense (about 2.7 times the
+    width) and of 16 experts of a quarter of that inner size, two a token by a table, beside a shared expert of that size."""
+    H = width // 64
+    inner = (width * 11 // 4 + 127) // 128 * 128
+    dense = {"ff": inner, "kind": "dense"}
+    moe = {"kind": "moe", "expert": {"ff": inner // 4}, "router": {"experts": 16, "top": 2}, "shared": {"ff": inner // 4}}
+    att = lambda mlp: {"type": "attention", "mlp": mlp,
+                       "mixer": {"dim": 64, "heads": H, "kv_heads": max(1, H // 4), "vdim": 64, "scale": 0.125, "softcap": 30.0,
+                                 "v_mix": True, "mask": {"size": 1024, "keep_first": 4},
+                                 "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0,
+                                                                                   "original": 1024}}}}
+    mem = lambda mlp: {"type": "mlstm", "mlp": mlp, "mixer": {"dim": 64, "heads": H // 2, "vdim": 128, "gate_cap": 15.0}}
+    layers = [f(moe if i % 2 else dense) for i, f in enumerate([att, mem, mem, att, mem] * 2)]
+    return {"architecture": "Fisesun", "vocab": vocab, "width": width, "embedding": {"scale": 2.0}, "norm": {"eps": 1e-5},
+            "logit_softcap": 30.0, "layers": layers}
+
+
+def run_fisesun(args):
+    """The same measurements as ``--only vobusun`` for the Fisesun design, beside Dalorax (the nearest design in the tree for its
+    attention and experts: windows with kept first positions, capped scores, norms on the sublayers' results) and Vobusun (the
+    nearest for its memories: retention with heads of the same size) at equal width and as many layers."""
+    vocab = 32000
+
+    def models(width):
+        fis = fisesun_config(width, vocab)
+        return len(fis["layers"]), [("fisesun", fis), ("dalorax", dalorax_config(width, vocab)),
+                                    ("vobusun", vobusun_config(width, vocab))]
+    run_beside(args, "fisesun_vs_dalorax", models)
+
+
 def run_vobusun(args):
     """The same measurements as ``--only zuluvik`` for the Vobusun design, beside Nufetar (the nearest design in the tree: a
     float32 stream, attention over latent rows in a window, a linear recurrence per head, dense feed-forwards) and Lelatar
@@ -897,9 +930,9 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration's 24 (0 = all)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--widths", default="", help="with --only lelatar / nufetar / dalorax / zuluvik / vobusun: the model widths to run, with commas (default 1024,2048)")
+    ap.add_argument("--widths", default="", help="with --only lelatar / nufetar / dalorax / zuluvik / vobusun / fisesun: the model widths to run, with commas (default 1024,2048)")
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "mixed", "timeline", "kernels", "yardstick",
-                                                   "lelatar", "nufetar", "dalorax", "zuluvik", "vobusun"],
+                                                   "lelatar", "nufetar", "dalorax", "zuluvik", "vobusun", "fisesun"],
                     help="run just this part and print its figures (decode / prefill: short runs for profiling; "
                          "mixed: 64 requests with prompts of 16..1024 tokens through the scheduler, 256-token portions "
                          "beside decoding requests; timeline: every kernel of one step with its start and end, "
@@ -909,7 +942,8 @@ def main():
                          "the Lelatar design at two widths beside GPT-2 of equal width and layer runs, with every kernel "
                          "of both against its roofline; nufetar: the same for the Nufetar design beside Lelatar; dalorax: the same for the Dalorax design "
                          "beside Nufetar; zuluvik: the same for the Zuluvik design beside Dalorax and Nufetar; "
-                         "vobusun: the same for the Vobusun design beside Nufetar and Lelatar)")
+                         "vobusun: the same for the Vobusun design beside Nufetar and Lelatar; fisesun: the same for the Fisesun design "
+                         "beside Dalorax and Vobusun)")
     ap.add_argument("--prefill-prompts", type=int, default=0,
                     help="with --only prefill: 1024-token prompts in the one step (default and the contract's figure: "
                          "2); with --only timeline: the timeline of such a step instead of a decode step")
@@ -939,6 +973,9 @@ def main():
         return 0
     if a.only == "vobusun":
         run_vobusun(a)
+        return 0
+    if a.only == "fisesun":
+        run_fisesun(a)
         return 0
     run_ours(a)
     return 0
