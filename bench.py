@@ -332,7 +332,9 @@ def kernel_table(calls, pk, mode, attention_bytes=0.0, attention_flops=0.0, reps
         graph = torch.cuda.CUDAGraph()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
-            for f, lib, fname, args, _ in launches:            # once eagerly
+            # the whole step first (a group replayed alone changes what the next one would read: a residual stream grows with
+            # every update), then the group once eagerly
+            for f, lib, fname, args, _ in list(calls) + list(launches):
                 f(*args[:-1], side.cuda_stream)
         side.synchronize()
         with torch.cuda.graph(graph, stream=side):

@@ -8,7 +8,8 @@
 //                  silu(g) BEFORE the statistics, mode 2 multiplies the normed value by silu(g).
 //                  x is float32 or has the activation dtype, which the result has.  No weight: the normed value as it is
 //                  (times the offset where there is one).  All arithmetic is float32.  Rows or parts of up to
-//                  512 columns without a weight, or in the activation dtype, take a kernel with a warp each.
+//                  512 columns without a weight, or in the activation dtype, take a kernel with a warp each; whole float32
+//                  rows with a weight per column one that keeps a row in registers.
 // residual_update  x[r, :] += scale * (f1(y1[r, :]) + f2(y2[r, :])),  f_i = rmsnorm with weight w_i over the
 //                  whole row, or the identity where w_i is null; y2 may be null.  Optionally a copy of the new
 //                  row in the activation dtype is left in `cast_out` for the products that read it next.
@@ -126,6 +127,48 @@ rmsnorm_parts_kernel(const TI* x, int ldx, const float* __restrict__ w, float of
   }
 }
 
+// Whole float32 rows with a weight per column, four columns a thread and step: the row stays in registers between the sum and
+// the result, the weights are asked for before the wait.  NV * 4 * blockDim.x columns at most.
+template <typename TO, int NV>
+__global__ void __launch_bounds__(512)
+rmsnorm_rows_kernel(const float* x, int ldx, const int* __restrict__ rows, int n_src_rows, const float* __restrict__ w, float offset,
+                    TO* __restrict__ out, int ldo, int D, float eps) {
+  __shared__ float red[33];
+  const int r = blockIdx.x;
+  const int src = rows ? rows[r] : r;
+  const bool there = src >= 0 && src < n_src_rows;
+  float wv[NV][4], v[NV][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 4;
+    if (c < D) load4(w + c, wv[i]);
+  }
+  pdl_wait();
+  pdl_trigger();
+  x = after_wait(x);
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[i][e] = 0.f;
+    if (c < D && there) load4(x + (size_t)src * ldx + c, v[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s = fmaf(v[i][e], v[i][e], s);
+  const float rinv = 1.f / sqrtf(block_sum(s, red) / (float)D + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 4;
+    if (c >= D) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[i][e] = v[i][e] * rinv * (offset + wv[i][e]);
+    store4(out + (size_t)r * ldo + c, v[i]);
+  }
+}
+
 // x_f32: x is float32 (else it has out_dtype); w may be null (the offset is then the factor).
 MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, int x_f32, const void* x, int ldx, const int* rows, int n_src_rows, const float* w,
                              float offset, int period, const void* gate, int ldg, int gate_mode, void* out, int ldo,
@@ -140,9 +183,28 @@ MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, int x_f32, const void* x, int ldx, c
   if (out_dtype != MLXB_F32 && out_dtype != MLXB_BF16) return mlxb_fail(MLXB_BAD_DTYPE, "rmsnorm: dtype code %d", out_dtype);
   const int Dg = D / groups;
   const int xb = (x_f32 || out_dtype == MLXB_F32) ? 16 : 8, ob = out_dtype == MLXB_F32 ? 16 : 8;   // bytes of four columns
-  // (weighted norms of float32 rows keep the block per row or part and its order of additions)
   const bool parts = (w == nullptr || (!x_f32 && out_dtype == MLXB_BF16)) && rows == nullptr && Dg % 4 == 0 && Dg <= 128 * RP_STEPS && ldx % 4 == 0 && ldo % 4 == 0 &&
                      (!gate || ldg % 4 == 0) && (uintptr_t)x % xb == 0 && ((uintptr_t)out | (uintptr_t)gate) % ob == 0;
+  if (x_f32 && w && groups == 1 && period == D && gate_mode == 0 && D % 4 == 0 && D <= 4 * 512 * 4 && ldx % 4 == 0 && ldo % 4 == 0 &&
+      (((uintptr_t)x | (uintptr_t)w) & 15) == 0 && (uintptr_t)out % ob == 0) {
+    int nt = 64;
+    while (nt < 512 && D / 4 > nt * 2) nt *= 2;
+    const int nv = (D / 4 + nt - 1) / nt;
+#define RMS_ROWS(TO, NV)                                                                                                \
+  launch_pdl(rmsnorm_rows_kernel<TO, NV>, dim3(R), dim3(nt), 0, stream, (const float*)x, ldx, rows, n_src_rows, w, offset, \
+             (TO*)out, ldo, D, eps)
+#define RMS_ROWS_NV(TO)               \
+  do {                                \
+    if (nv <= 1) RMS_ROWS(TO, 1);     \
+    else if (nv <= 2) RMS_ROWS(TO, 2); \
+    else RMS_ROWS(TO, 4);             \
+  } while (0)
+    if (out_dtype == MLXB_F32) RMS_ROWS_NV(float);
+    else RMS_ROWS_NV(__nv_bfloat16);
+#undef RMS_ROWS_NV
+#undef RMS_ROWS
+    return mlxb_check_launch("rmsnorm");
+  }
   const int threads = parts ? 256 : (Dg >= 2048 ? 256 : (Dg >= 512 ? 128 : (Dg >= 128 ? 64 : 32)));
   const dim3 grid = parts ? dim3((unsigned)(((long long)R * groups + 7) / 8)) : dim3(R, groups);
 #define RMS_GO(TI, TO)                                                                                                  if (parts)                                                                                                              launch_pdl(rmsnorm_parts_kernel<TI, TO>, grid, dim3(threads), 0, stream, (const TI*)x, ldx, w, offset, period,                   (const TO*)gate, ldg, gate_mode, (TO*)out, ldo, R, Dg, groups, eps);                                     else                                                                                                                    launch_pdl(rmsnorm_kernel<TI, TO>, grid, dim3(threads), 0, stream, (const TI*)x, ldx, rows, n_src_rows, w, offset,                period, (const TO*)gate, ldg, gate_mode, (TO*)out, ldo, D, groups, eps)
