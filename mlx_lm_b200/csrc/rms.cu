@@ -8,8 +8,8 @@
 //                  silu(g) BEFORE the statistics, mode 2 multiplies the normed value by silu(g).
 //                  x is float32 or has the activation dtype, which the result has.  No weight: the normed value as it is
 //                  (times the offset where there is one).  All arithmetic is float32.  Rows or parts of up to
-//                  512 columns without a weight, or in the activation dtype, take a kernel with a warp each; whole float32
-//                  rows with a weight per column one that keeps a row in registers.
+//                  512 columns without a weight, or in the activation dtype, take a kernel with a warp each.
+// rmsnorm_rows     the same for whole float32 rows with a weight per column, a row kept in registers.
 // residual_update  x[r, :] += scale * (f1(y1[r, :]) + f2(y2[r, :])),  f_i = rmsnorm with weight w_i over the
 //                  whole row, or the identity where w_i is null; y2 may be null.  Optionally a copy of the new
 //                  row in the activation dtype is left in `cast_out` for the products that read it next.
@@ -183,28 +183,9 @@ MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, int x_f32, const void* x, int ldx, c
   if (out_dtype != MLXB_F32 && out_dtype != MLXB_BF16) return mlxb_fail(MLXB_BAD_DTYPE, "rmsnorm: dtype code %d", out_dtype);
   const int Dg = D / groups;
   const int xb = (x_f32 || out_dtype == MLXB_F32) ? 16 : 8, ob = out_dtype == MLXB_F32 ? 16 : 8;   // bytes of four columns
+  // (weighted norms of float32 rows keep the block per row or part and its order of additions)
   const bool parts = (w == nullptr || (!x_f32 && out_dtype == MLXB_BF16)) && rows == nullptr && Dg % 4 == 0 && Dg <= 128 * RP_STEPS && ldx % 4 == 0 && ldo % 4 == 0 &&
                      (!gate || ldg % 4 == 0) && (uintptr_t)x % xb == 0 && ((uintptr_t)out | (uintptr_t)gate) % ob == 0;
-  if (x_f32 && w && groups == 1 && period == D && gate_mode == 0 && D % 4 == 0 && D <= 4 * 512 * 4 && ldx % 4 == 0 && ldo % 4 == 0 &&
-      (((uintptr_t)x | (uintptr_t)w) & 15) == 0 && (uintptr_t)out % ob == 0) {
-    int nt = 64;
-    while (nt < 512 && D / 4 > nt * 2) nt *= 2;
-    const int nv = (D / 4 + nt - 1) / nt;
-#define RMS_ROWS(TO, NV)                                                                                                \
-  launch_pdl(rmsnorm_rows_kernel<TO, NV>, dim3(R), dim3(nt), 0, stream, (const float*)x, ldx, rows, n_src_rows, w, offset, \
-             (TO*)out, ldo, D, eps)
-#define RMS_ROWS_NV(TO)               \
-  do {                                \
-    if (nv <= 1) RMS_ROWS(TO, 1);     \
-    else if (nv <= 2) RMS_ROWS(TO, 2); \
-    else RMS_ROWS(TO, 4);             \
-  } while (0)
-    if (out_dtype == MLXB_F32) RMS_ROWS_NV(float);
-    else RMS_ROWS_NV(__nv_bfloat16);
-#undef RMS_ROWS_NV
-#undef RMS_ROWS
-    return mlxb_check_launch("rmsnorm");
-  }
   const int threads = parts ? 256 : (Dg >= 2048 ? 256 : (Dg >= 512 ? 128 : (Dg >= 128 ? 64 : 32)));
   const dim3 grid = parts ? dim3((unsigned)(((long long)R * groups + 7) / 8)) : dim3(R, groups);
 #define RMS_GO(TI, TO)                                                                                                  if (parts)                                                                                                              launch_pdl(rmsnorm_parts_kernel<TI, TO>, grid, dim3(threads), 0, stream, (const TI*)x, ldx, w, offset, period,                   (const TO*)gate, ldg, gate_mode, (TO*)out, ldo, R, Dg, groups, eps);                                     else                                                                                                                    launch_pdl(rmsnorm_kernel<TI, TO>, grid, dim3(threads), 0, stream, (const TI*)x, ldx, rows, n_src_rows, w, offset,                period, (const TO*)gate, ldg, gate_mode, (TO*)out, ldo, D, groups, eps)
@@ -213,6 +194,35 @@ MLXB_EXPORT int mlxb_rmsnorm(int out_dtype, int x_f32, const void* x, int ldx, c
   else { RMS_GO(__nv_bfloat16, __nv_bfloat16); }
 #undef RMS_GO
   return mlxb_check_launch("rmsnorm");
+}
+
+// x: float32 rows at stride ldx, whole groups of four columns, 16-byte aligned, at most 8192 wide; rows: int32 [R] or null; w:
+// float32 [D]; out: [R, D] of out_dtype.
+MLXB_EXPORT int mlxb_rmsnorm_rows(int out_dtype, const float* x, int ldx, const int* rows, int n_src_rows, const float* w,
+                                  float offset, void* out, int ldo, int R, int D, float eps, cudaStream_t stream) {
+  if (R <= 0) return 0;
+  const int ob = out_dtype == MLXB_F32 ? 16 : 8;
+  if (D <= 0 || D % 4 || D > 4 * 512 * 4 || ldx % 4 || ldo % 4 || ldx < D || ldo < D || !w || (((uintptr_t)x | (uintptr_t)w) & 15) ||
+      (uintptr_t)out % ob)
+    return mlxb_fail(MLXB_BAD_ARG, "rmsnorm_rows: width %d, strides %d / %d", D, ldx, ldo);
+  int threads = 64;
+  while (threads < 512 && D / 4 > threads * 2) threads *= 2;
+  const int nv = (D / 4 + threads - 1) / threads;
+#define RMS_ROWS(TO, NV)                                                                                                \
+  launch_pdl(rmsnorm_rows_kernel<TO, NV>, dim3(R), dim3(threads), 0, stream, x, ldx, rows, n_src_rows, w, offset, (TO*)out, ldo, \
+             D, eps)
+#define RMS_ROWS_NV(TO)                \
+  do {                                 \
+    if (nv <= 1) RMS_ROWS(TO, 1);      \
+    else if (nv <= 2) RMS_ROWS(TO, 2); \
+    else RMS_ROWS(TO, 4);              \
+  } while (0)
+  if (out_dtype == MLXB_F32) RMS_ROWS_NV(float);
+  else if (out_dtype == MLXB_BF16) RMS_ROWS_NV(__nv_bfloat16);
+  else return mlxb_fail(MLXB_BAD_DTYPE, "rmsnorm_rows: dtype code %d", out_dtype);
+#undef RMS_ROWS_NV
+#undef RMS_ROWS
+  return mlxb_check_launch("rmsnorm_rows");
 }
 
 template <typename TO>

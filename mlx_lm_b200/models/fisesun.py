@@ -159,7 +159,7 @@ def build(args: ModelArgs) -> ModelDescription:
         blocks.append(OutputNormBlock(RMSNorm(f"{p}.norm1", D, eps), _mixer(f"{p}.mix", D, spec, eps, value_mix), norm_2, ff))
     return ModelDescription(
         model_type="fisesun", width=D, vocab_size=args.vocab, embedding=embed, position=None, blocks=blocks,
-        final_norm=RMSNorm("final.norm", D, eps),
+        final_norm=RMSNorm("final.norm", D, eps, in_registers=True),
         head=OutputHead(args.vocab, D, name="head", weight_suffix="", init=Init(0.0, D ** -0.5), softcap=args.logit_softcap),
         args=args)
 

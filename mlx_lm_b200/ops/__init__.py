@@ -825,6 +825,29 @@ def rmsnorm(x, weight, out, eps: float, stream, offset: float = 0.0, groups: int
           groups, float(eps), stream)
 
 
+def rmsnorm_rows_supported(x, weight, out) -> bool:
+    """Whether ``rmsnorm_rows`` takes these rows (whole groups of four columns, aligned, at most 8192 wide)."""
+    D = out.shape[1]
+    return (x.dtype == torch.float32 and D % 4 == 0 and D <= 8192 and x.stride(0) % 4 == 0 and out.stride(0) % 4 == 0
+            and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0)
+
+
+def rmsnorm_rows(x, weight, out, eps: float, stream, offset: float = 0.0, rows=None) -> None:
+    """``rmsnorm`` of whole float32 rows with a weight per column and neither parts nor a gate, a row kept in registers between
+    its sum and the result (another order of additions)."""
+    _need(x, torch.float32, "rmsnorm_rows x")
+    _need(weight, torch.float32, "rmsnorm_rows weight")
+    R, D = out.shape
+    if rows is not None:
+        _need(rows, torch.int32, "rmsnorm_rows rows")
+    if x.shape[1] != D or weight.numel() != D or (rows.numel() if rows is not None else x.shape[0]) != R:
+        raise KernelError(f"rmsnorm_rows: x {tuple(x.shape)}, weight of {weight.numel()}, out {tuple(out.shape)}")
+    _call("rms", "mlxb_rmsnorm_rows", [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_int,
+                                       c_float, c_void_p],
+          dtype_code(out.dtype), _p(x), _rows(x, "rmsnorm_rows x"), _p(rows), x.shape[0], _p(weight), float(offset), _p(out),
+          _rows(out, "rmsnorm_rows out"), R, D, float(eps), stream)
+
+
 _RESUP_ARGS = [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int,
                c_int, c_int, c_void_p]
 

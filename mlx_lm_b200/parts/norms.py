@@ -45,13 +45,14 @@ class LayerNorm(Norm):
 
 class RMSNorm(Norm):
     """``x / sqrt(mean(x^2) + eps) * (offset + weight)`` over float32 rows, result in the run's dtype.
-    ``offset = 1``: the weight is stored as its distance from one; ``offset = 0``: as it is."""
+    ``offset = 1``: the weight is stored as its distance from one; ``offset = 0``: as it is.  ``in_registers``: rows go through
+    the kernel that reads them once, where their width allows it (results differ in the last bits)."""
     replayable = True
     kernel_libs = ("rms",)
 
     def __init__(self, name: str, width: int, eps: float, offset: float = 0.0, weight_suffix: str = "",
-                 init: Optional[Init] = None):
-        self.name, self.width, self.eps, self.offset = name, width, float(eps), float(offset)
+                 init: Optional[Init] = None, in_registers: bool = False):
+        self.name, self.width, self.eps, self.offset, self.in_registers = name, width, float(eps), float(offset), in_registers
         self.weight_name = name + weight_suffix
         self.init = init if init is not None else Init(1.0 - self.offset, 0.1)
         self.weight = self._plain = None
@@ -66,7 +67,10 @@ class RMSNorm(Norm):
         n = x.shape[0] if rows is None else rows.numel()
         out = ctx.ws.get(tag, n, self.width, ctx.dtype)
         ops.label(self.name, 4.0 * n * self.width, (4.0 + out.element_size()) * n * self.width)
-        ops.rmsnorm(x, self.weight, out, self.eps, ctx.stream, offset=self.offset, rows=rows)
+        if self.in_registers and ops.rmsnorm_rows_supported(x, self.weight, out):
+            ops.rmsnorm_rows(x, self.weight, out, self.eps, ctx.stream, offset=self.offset, rows=rows)
+        else:
+            ops.rmsnorm(x, self.weight, out, self.eps, ctx.stream, offset=self.offset, rows=rows)
         return out
 
     def rms_args(self):

@@ -237,6 +237,23 @@ def test_stream_update_through_a_norm_of_a_sum(act, D, terms, extra):
     assert torch.equal(again.cpu(), x.cpu())
 
 
+@pytest.mark.parametrize("act", ACT)
+@pytest.mark.parametrize("D", [64, 100, 1032, 2048, 8192])
+def test_rms_norm_of_rows_kept_in_registers(act, D):
+    from mlx_lm_b200 import ops
+    torch.manual_seed(D)
+    x, w, rows = torch.randn(9, D) * 3, torch.randn(D), [7, 0, 0, 8, -1]
+    for offset in (0.0, 1.0):
+        want = plain.rms(x.double(), 1e-5) * (offset + w.double())
+        tol = (2e-6 if act == torch.float32 else 5e-3) * float(want.abs().max())
+        out, picked = torch.zeros(9, D, dtype=act, device=DEV), torch.full((5, D), 4.0, dtype=act, device=DEV)
+        assert ops.rmsnorm_rows_supported(x.to(DEV), w.to(DEV), out)
+        ops.rmsnorm_rows(x.to(DEV), w.to(DEV), out, 1e-5, stream(), offset=offset)
+        assert float((out.cpu().double() - want).abs().max()) < tol
+        ops.rmsnorm_rows(x.to(DEV), w.to(DEV), picked, 1e-5, stream(), offset=offset, rows=i32(rows))
+        assert torch.equal(picked.cpu()[:4], out.cpu()[rows[:4]]) and float(picked[4].float().abs().max()) == 0.0
+
+
 @pytest.mark.parametrize("T,E,top,rows", [(5, 3, 1, 4), (700, 16, 2, 128), (64, 9, 4, 16), (1, 1, 1, 64), (2000, 40, 3, 64)])
 def test_plan_of_experts_named_by_a_table(T, E, top, rows):
     from mlx_lm_b200 import ops
