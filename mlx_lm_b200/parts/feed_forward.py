@@ -146,7 +146,9 @@ class ExpertsMLP(FeedForward):
         self.correction = None
         self.table_name, self.table_vocab, self.table = f"{name}.{table_name}", int(table_vocab), None
         self.router = None
-        if not table_vocab:
+        if table_vocab:
+            self.kernel_libs = ("moe", "moe_tcgen05")      # the sum over a token's experts is the block's
+        else:
             self.router = Linear(f"{name}.{router_name}", width, n_outputs, bias=False, weight_suffix="", init=router_init)
         self.names = [(f"{name}.{expert_prefix}{e}.{gate_name}", f"{name}.{expert_prefix}{e}.{up_name}",
                        f"{name}.{expert_prefix}{e}.{down_name}") for e in range(n_experts)]
@@ -251,7 +253,7 @@ class ExpertsMLP(FeedForward):
         return y, sel_e, sel_w
 
     def forward(self, ctx, x, residual):
-        if self.table_vocab and self.top != 1:
+        if self.table_vocab:
             raise ops.KernelError(f"{self.name}: experts out of a table come with a factor (summands)")
         y, sel_e, sel_w = self._experts(ctx, x)
         terms = self.top
