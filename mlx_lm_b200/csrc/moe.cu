@@ -214,6 +214,8 @@ struct MoeTable {
 
 // sorted [S]; tile_info [max_tiles][3]; n_tiles [1].  Shared memory: 3 E + 1 ints.  EARLY: the experts follow from the step's
 // inputs and are counted before the wait for the kernel before.
+constexpr int MP_KEEP = 4;
+
 template <typename Source, bool EARLY>
 __global__ void moe_plan_kernel(Source expert_of, int S, int E, int tile_rows, int max_tiles,
                                 int* __restrict__ sorted, int* __restrict__ tile_info, int* __restrict__ n_tiles) {
@@ -228,7 +230,16 @@ __global__ void moe_plan_kernel(Source expert_of, int S, int E, int tile_rows, i
     expert_of.arrived();
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < S; i += blockDim.x) {
+  int mine[MP_KEEP];            // the experts of this thread's first slots, looked up once
+#pragma unroll
+  for (int j = 0; j < MP_KEEP; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    mine[j] = i < S ? expert_of(i) : -1;
+  }
+#pragma unroll
+  for (int j = 0; j < MP_KEEP; ++j)
+    if (mine[j] >= 0 && mine[j] < E) atomicAdd(&cnt[mine[j]], 1);
+  for (int i = threadIdx.x + MP_KEEP * blockDim.x; i < S; i += blockDim.x) {
     const int e = expert_of(i);
     if (e >= 0 && e < E) atomicAdd(&cnt[e], 1);
   }
@@ -252,7 +263,10 @@ __global__ void moe_plan_kernel(Source expert_of, int S, int E, int tile_rows, i
     n_tiles[0] = nt;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < S; i += blockDim.x) {
+#pragma unroll
+  for (int j = 0; j < MP_KEEP; ++j)
+    if (mine[j] >= 0 && mine[j] < E) sorted[off[mine[j]] + atomicAdd(&cur[mine[j]], 1)] = threadIdx.x + j * blockDim.x;
+  for (int i = threadIdx.x + MP_KEEP * blockDim.x; i < S; i += blockDim.x) {
     const int e = expert_of(i);
     if (e >= 0 && e < E) sorted[off[e] + atomicAdd(&cur[e], 1)] = i;
   }

@@ -229,7 +229,7 @@ class ExpertsMLP(FeedForward):
         tiles = ctx.ws.flat("moe_tiles", 3 * max_tiles + 1, torch.int32)
         n_tiles = tiles[3 * max_tiles:]
         if self.table_vocab:
-            ops.label(self.name + ".plan", 0.0, 4.0 * T + 8.0 * S)
+            ops.label(self.name + ".plan", 0.0, 8.0 * T + 8.0 * S)
             ops.moe_plan_table(ctx.tokens, ctx.token_req, self.table, T, E, rows, order, tiles, n_tiles, ctx.status, ctx.stream)
         else:
             ops.moe_plan(sel_e, S, E, rows, order, tiles, n_tiles, ctx.stream)
