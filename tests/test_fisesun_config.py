@@ -146,15 +146,15 @@ def test_random_weights_give_a_working_plain_model():
 def test_frequencies_by_wavelength():
     """Short wavelengths keep their frequency, long ones are stretched, those between are blended; the framework's table and
     the plain one agree."""
-    rot = {"dims": 64, "base": 10000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 512}}
+    rot = {"dims": 64, "base": 10000.0, "scaling": {"factor": 6.0, "low": 1.5, "high": 5.0, "original": 700}}
     f = plain.frequencies(dict(rot, scaling=None))
     got = plain.frequencies(rot)
     length = 2 * math.pi / f
-    short, long_ = length < 512 / 4.0, length > 512 / 1.0
+    short, long_ = length < 700 / 5.0, length > 700 / 1.5
     assert bool(short.any()) and bool(long_.any()) and bool((~short & ~long_).any())
-    assert torch.equal(got[short], f[short]) and torch.allclose(got[long_], f[long_] / 8.0)
+    assert torch.equal(got[short], f[short]) and torch.allclose(got[long_], f[long_] / 6.0)
     mid = ~short & ~long_
-    assert bool((got[mid] < f[mid]).all()) and bool((got[mid] > f[mid] / 8.0).all())
+    assert bool((got[mid] < f[mid]).all()) and bool((got[mid] > f[mid] / 6.0).all())
     for r in (rot, {"dims": 10, "base": 50.0, "scaling": {"factor": 3.0, "low": 2.0, "high": 2.0, "original": 40}},
               {"dims": 6, "base": 1e6, "scaling": {"factor": 1.0, "low": 0.5, "high": 7.0, "original": 1000}}):
         mine, factor = rotation_frequencies(r["dims"], r["base"], r["scaling"])
